@@ -182,6 +182,21 @@ _CUDA_SIG = {
     "ggb_op_hyper_mix": (i32, [i32, vp, vp, vp, vp, vp, i32, vp, vp, f32, i64, i64, vp, vp, vp]),
     "ggb_op_act_rows": (i32, [i32, vp, i64, i64, i64, i32, vp]),
     "ggb_op_linear_relu2": (i32, [i32, vp, i64, i64, vp, i64, i64, vp, vp]),
+    "ggb_op_shift_norm": (i32, [i32, vp, vp, vp, vp, vp, vp, vp, vp, f32, vp, vp, i64, i64, vp, vp, vp, vp]),
+    "ggb_op_linear_pair": (i32, [i32, vp, i64, i64, vp, i64, vp, i64, i64, vp, i64, i64, vp, i64, vp, f32, f32, vp, i64]),
+    "ggb_op_xielu_rows": (i32, [i32, vp, i64, f32, f32, vp]),
+    "ggb_rglru_history_rows": (i32, [i32]), "ggb_rglru_step_form": (i32, [i64, i32]), "ggb_rglru_split_fits": (i32, [i32, i64, i32]),
+    "ggb_op_rglru_step": (i32, [i32, vp, vp, i64, i64, i32, i32, vp, vp, i32, vp, vp, vp, vp, vp, vp, vp, vp, vp]),
+    "ggb_op_rglru_conv": (i32, [vp, i64, i64, i32, i32, vp, vp, i32, vp, vp, vp, vp, vp, vp]),
+    "ggb_op_rglru_gates": (i32, [i32, vp, vp, vp, i64, i32, i32, vp, vp, vp]),
+    "ggb_op_rglru_scan": (i32, [i32, vp, vp, vp, i64, i64, i32, i32, vp, vp, vp, vp, vp]),
+    "ggb_op_masked_attn_keep": (i32, [i32, vp, vp, vp, i32, vp, i64, i32, i32, i32, i32, i64, i64, f32, vp, vp]),
+    "ggb_op_diff_qkv_store": (i32, [i32, vp, vp, vp, i64, i64, i32, i32, i32, i32, i32, i32, vp, f32, vp, vp, i32, vp, vp]),
+    "ggb_op_diff_attn": (i32, [i32, vp, vp, vp, i32, vp, i64, i32, i32, i32, i32, i64, i64, f32, f32, f32, f32, vp, i64, vp, vp]),
+    "ggb_op_latent_prep": (i32, [i32, vp, i32, vp, vp, vp, i64, i64, i32, i32, i32, i32, vp, f32, vp, vp, vp, i32, vp]),
+    "ggb_op_latent_q_absorb_halves": (i32, [i32, vp, i64, i64, i32, i32, i32, i32, vp, vp, vp, i32, f32, vp]),
+    "ggb_op_latent_expand_rot": (i32, [i32, vp, vp, i32, i64, i64, i32, i32, i32, i32, i32, vp, vp, vp, vp, i64]),
+    "ggb_op_latent_q_rotate": (i32, [vp, i64, i64, i32, i32, i32, i32, i32, vp, vp, f32, vp]),
     "ggb_op_hyper_mix_moe": (i32, [i32, vp, vp, vp, vp, vp, i64, i32, i32, i32, vp, vp, vp, i32, vp, vp, f32, i64, i64, vp, vp, vp]),
     "ggb_comm_unique_id": (i32, [vp]), "ggb_comm_init": (i32, [vp, i32, i32]), "ggb_comm_destroy": (i32, []),
     "ggb_comm_rank": (i32, []), "ggb_comm_size": (i32, []), "ggb_op_allgather": (i32, [vp, vp, sz]),
@@ -224,6 +239,7 @@ _HOST_SIG = {
     "bg_config_probe": (i32, [C.c_char_p, P(i64)]),
     "dl_config_probe": (i32, [C.c_char_p, P(i64)]),
     "kb_config_probe": (i32, [C.c_char_p, P(i64)]),
+    "tz_config_probe": (i32, [C.c_char_p, P(i64)]),
     "st_probe": (i32, [C.c_char_p, C.c_char_p, P(i64), P(i64), C.c_char_p, i32, P(i64)]),
     "mul_mat": (None, [i64, i64, i64, i64, i64, i64, i64, sz, i64, vp, vp, vp, vp, i32, vp]),
     "init_cuda_offload": (i32, [i32]),

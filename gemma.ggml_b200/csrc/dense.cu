@@ -19,20 +19,12 @@ namespace {
 // 16-byte loads and keeps T accumulators.  HBM-bound (decode).
 constexpr int kVecT = 8;
 
-// ACT 1: the output is relu(.)^2 in the matrices' type (c_act) instead of fp32 (c)
-template <typename E, int TT, int ACT = 0>
-__global__ void __launch_bounds__(256) linear_vec_kernel(const E *__restrict__ w, int64_t N, int64_t K, const E *__restrict__ a,
-                                                         int64_t lda, float *__restrict__ c, int64_t ldc, E *__restrict__ c_act = nullptr) {
+// acc[t] = the lane's share of row wr (K numbers) against TT rows of a
+template <typename E, int TT>
+__device__ __forceinline__ void vec_row_dot(const E *__restrict__ wr, const E *__restrict__ a, int64_t lda, int64_t K, bool vec, int lane, float (&acc)[TT]) {
     constexpr int VE = 16 / (int)sizeof(E); // elements per 16-byte load
-    const int lane = threadIdx.x & 31;
-    const int64_t n = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (n >= N) return;
-    float acc[TT];
 #pragma unroll
     for (int t = 0; t < TT; t++) acc[t] = 0.f;
-    const E *wr = w + n * K;
-    const bool vec = (K % VE == 0) && ((reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(a)) % 16 == 0) &&
-                     (lda % VE == 0);
     if (vec) {
 #pragma unroll 4
         for (int64_t k = (int64_t)lane * VE; k < K; k += 32 * VE) { // several 16-byte loads of the row in flight
@@ -56,6 +48,20 @@ __global__ void __launch_bounds__(256) linear_vec_kernel(const E *__restrict__ w
             for (int t = 0; t < TT; t++) acc[t] = fmaf(wf, to_f32(a[t * lda + k]), acc[t]);
         }
     }
+}
+
+// ACT 1: the output is relu(.)^2 in the matrices' type (c_act) instead of fp32 (c)
+template <typename E, int TT, int ACT = 0>
+__global__ void __launch_bounds__(256) linear_vec_kernel(const E *__restrict__ w, int64_t N, int64_t K, const E *__restrict__ a,
+                                                         int64_t lda, float *__restrict__ c, int64_t ldc, E *__restrict__ c_act = nullptr) {
+    constexpr int VE = 16 / (int)sizeof(E);
+    const int lane = threadIdx.x & 31;
+    const int64_t n = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (n >= N) return;
+    float acc[TT];
+    const bool vec = (K % VE == 0) && ((reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(a)) % 16 == 0) &&
+                     (lda % VE == 0);
+    vec_row_dot<E, TT>(w + n * K, a, lda, K, vec, lane, acc);
 #pragma unroll
     for (int t = 0; t < TT; t++) {
         const float s = warp_sum_f32(acc[t]);
@@ -184,10 +190,6 @@ __global__ void glu_clamp_kernel(const float *__restrict__ gu, int64_t F, int64_
     const float g = fminf(gu[t * 2 * F + f], limit);
     const float u = fminf(fmaxf(gu[t * 2 * F + F + f], -limit), limit);
     y[i] = from_f32<E>(g / (1.0f + expf(-alpha * g)) * (u + 1.0f));
-}
-
-__device__ __forceinline__ float gelu_tanh_f32(float z) {
-    return 0.5f * z * (1.0f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
 }
 
 // x <- x + a (+ f); then, with a side input, x <- x + rms(y) * nw, y = proj (gelu_tanh(gate x) * e), e = the token's
@@ -1029,6 +1031,261 @@ int ggb_op_act_rows(int dt, const float *x, int64_t ldx, int64_t T, int64_t F, i
     else act_rows_kernel<<<blocks, 256, 0, ggb_cuda_stream()>>>(x, ldx, T, F, act, (float *)y);
     GGB_LAUNCH_CHECK();
     return GGB_OK;
+}
+
+} // extern "C"
+
+// ------------------------------------------------------------------------------------------------ parallel sublayers: token shift, two products at once, xIELU
+namespace {
+
+struct xielu_args {
+    float ap = 0.f, an = 0.f; // the positive and the negative side's factor, after their softplus
+};
+// z > 0: ap z^2 + z / 2; z <= 0: an (exp(z) - 1 - z) + z / 2
+__device__ __forceinline__ float xielu_f32(float z, const xielu_args &x) {
+    return z > 0.f ? fmaf(x.ap * z, z, 0.5f * z) : fmaf(x.an, expm1f(z) - z, 0.5f * z);
+}
+
+template <typename E>
+__global__ void xielu_rows_kernel(const float *__restrict__ x, int64_t n, xielu_args xa, E *__restrict__ y) {
+    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) y[i] = from_f32<E>(xielu_f32(x[i], xa));
+}
+
+// one of two mat-vecs that share a launch
+template <typename E> struct vec_half {
+    const E *w, *a;
+    int64_t N, K, lda, ldc;
+    float *c;  // fp32 output, or
+    E *c_act;  // the output after the activation, in the matrices' type
+    xielu_args act;
+    int vec;
+};
+
+// the first `blocks1` CTAs take the rows of h1, the others those of h2
+template <typename E, int TT>
+__global__ void __launch_bounds__(256) linear_pair_kernel(vec_half<E> h1, vec_half<E> h2, int blocks1) {
+    const int lane = threadIdx.x & 31;
+    const bool first = (int)blockIdx.x < blocks1;
+    const vec_half<E> &h = first ? h1 : h2;
+    const int64_t n = (int64_t)(first ? blockIdx.x : blockIdx.x - blocks1) * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (n >= h.N) return;
+    float acc[TT];
+    vec_row_dot<E, TT>(h.w + n * h.K, h.a, h.lda, h.K, h.vec != 0, lane, acc);
+#pragma unroll
+    for (int t = 0; t < TT; t++) {
+        const float s = warp_sum_f32(acc[t]);
+        if (lane == 0) {
+            if (h.c_act) h.c_act[t * h.ldc + n] = from_f32<E>(xielu_f32(s, h.act));
+            else h.c[t * h.ldc + n] = s;
+        }
+    }
+}
+
+template <typename E>
+vec_half<E> make_half(const void *w, int64_t N, int64_t K, const void *a, int64_t lda, float *c, void *c_act, int64_t ldc, xielu_args act) {
+    constexpr int VE = 16 / (int)sizeof(E);
+    const int vec = K % VE == 0 && lda % VE == 0 && (((uintptr_t)w | (uintptr_t)a) & 15) == 0;
+    return vec_half<E>{(const E *)w, (const E *)a, N, K, lda, ldc, c, (E *)c_act, act, vec};
+}
+
+template <typename E>
+int linear_pair_launch(const vec_half<E> &h1, const vec_half<E> &h2, int64_t T) {
+    const int blocks1 = (int)((h1.N + 7) / 8);
+    const unsigned grid = (unsigned)(blocks1 + (h2.N + 7) / 8);
+    switch ((int)T) {
+#define PAIR_CASE(TT) case TT: linear_pair_kernel<E, TT><<<grid, 256, 0, ggb_cuda_stream()>>>(h1, h2, blocks1); break;
+        PAIR_CASE(1) PAIR_CASE(2) PAIR_CASE(3) PAIR_CASE(4) PAIR_CASE(5) PAIR_CASE(6) PAIR_CASE(7) PAIR_CASE(8)
+#undef PAIR_CASE
+    }
+    GGB_LAUNCH_CHECK();
+    return GGB_OK;
+}
+
+// The pass between two layers whose sublayers run side by side.  A CTA takes NT consecutive tokens:
+//   x' = x + (a * ls_a + b * ls_b)       the layer's two outputs, each with a weight per channel (a / b may be null)
+//   h  = x' / rms(x') * nw               in dt (h) and, per channel, blended with the token before: hs = h + (h_before - h) * mu
+// The token before the CTA's first one is computed again from the inputs (x' goes to another buffer than x), the one before the
+// portion comes from `prev` (fp32 [W], the sequence's state), which CTA 0 then replaces by the portion's last h.
+// table / ids instead of x: the residual starts as the token's embedding row.  rows: only those tokens, h only.
+template <typename E>
+struct shift_norm_args {
+    const float *x;
+    const E *table;
+    const int32_t *ids;
+    const float *a, *ls_a, *b, *ls_b, *nw, *mu;
+    float eps;
+    int64_t W, T;
+    const int32_t *rows;
+    float *prev, *x_out;
+    E *h, *hs;
+};
+
+template <typename E, int V, int TB>
+__global__ void __launch_bounds__(TB) shift_norm_kernel(shift_norm_args<E> p, int nt) {
+    extern __shared__ __align__(16) float sn_smem[]; // [W] the row, [W] the normed row before it
+    __shared__ float red[32];
+    float *cur = sn_smem, *before = sn_smem + p.W;
+    const int64_t W = p.W;
+    // x' of token t into `cur` (and x_out when asked); returns 1 / rms
+    auto row = [&](int64_t t, int64_t out_row, bool store) -> float {
+        float ss = 0.f;
+        const E *er = p.table ? p.table + (int64_t)p.ids[t] * W : nullptr;
+        for (int64_t i = (int64_t)threadIdx.x * V; i < W; i += (int64_t)TB * V) {
+            float x[V], ya[V], yb[V];
+            if (V == 4) {
+                if (er) {
+#pragma unroll
+                    for (int c = 0; c < V; c++) x[c] = to_f32(er[i + c]);
+                } else {
+                    const float4 v = *reinterpret_cast<const float4 *>(p.x + t * W + i);
+                    x[0] = v.x, x[1 % V] = v.y, x[2 % V] = v.z, x[3 % V] = v.w;
+                }
+                if (p.a) {
+                    const float4 v = *reinterpret_cast<const float4 *>(p.a + t * W + i), l = *reinterpret_cast<const float4 *>(p.ls_a + i);
+                    ya[0] = v.x * l.x, ya[1 % V] = v.y * l.y, ya[2 % V] = v.z * l.z, ya[3 % V] = v.w * l.w;
+                }
+                if (p.b) {
+                    const float4 v = *reinterpret_cast<const float4 *>(p.b + t * W + i), l = *reinterpret_cast<const float4 *>(p.ls_b + i);
+                    yb[0] = v.x * l.x, yb[1 % V] = v.y * l.y, yb[2 % V] = v.z * l.z, yb[3 % V] = v.w * l.w;
+                }
+            } else {
+                x[0] = er ? to_f32(er[i]) : p.x[t * W + i];
+                if (p.a) ya[0] = p.a[t * W + i] * p.ls_a[i];
+                if (p.b) yb[0] = p.b[t * W + i] * p.ls_b[i];
+            }
+#pragma unroll
+            for (int c = 0; c < V; c++) {
+                if (p.a) x[c] += p.b ? ya[c] + yb[c] : ya[c];
+                cur[i + c] = x[c];
+                ss = fmaf(x[c], x[c], ss);
+            }
+            if (store) {
+                if (V == 4) *reinterpret_cast<float4 *>(p.x_out + out_row * W + i) = make_float4(x[0], x[1 % V], x[2 % V], x[3 % V]);
+                else p.x_out[out_row * W + i] = x[0];
+            }
+        }
+        if (!p.nw) return 0.f;
+        return 1.0f / sqrtf(block_sum_any(ss, red) / (float)W + p.eps);
+    };
+    // every thread owns the same columns in every loop below: nothing but the root mean square crosses threads
+    if (p.rows) {
+        const int64_t o = blockIdx.x;
+        const float r = row(p.rows[o], o, false);
+        for (int64_t i = (int64_t)threadIdx.x * V; i < W; i += (int64_t)TB * V)
+#pragma unroll
+            for (int c = 0; c < V; c++) p.h[o * W + i + c] = from_f32<E>(cur[i + c] * r * p.nw[i + c]);
+        return;
+    }
+    const int64_t t0 = (int64_t)blockIdx.x * nt, t1 = min(p.T, t0 + nt);
+    if (p.mu) {
+        const float r = t0 > 0 ? row(t0 - 1, 0, false) : 0.f;
+        for (int64_t i = (int64_t)threadIdx.x * V; i < W; i += (int64_t)TB * V)
+#pragma unroll
+            for (int c = 0; c < V; c++) before[i + c] = t0 > 0 ? cur[i + c] * r * p.nw[i + c] : p.prev[i + c];
+    }
+    for (int64_t t = t0; t < t1; t++) {
+        const float r = row(t, t, p.x_out != nullptr);
+        if (!p.nw) continue;
+        for (int64_t i = (int64_t)threadIdx.x * V; i < W; i += (int64_t)TB * V) {
+#pragma unroll
+            for (int c = 0; c < V; c++) {
+                const float h = cur[i + c] * r * p.nw[i + c];
+                if (p.h) p.h[t * W + i + c] = from_f32<E>(h);
+                if (p.mu) {
+                    p.hs[t * W + i + c] = from_f32<E>(fmaf(before[i + c] - h, p.mu[i + c], h));
+                    before[i + c] = h;
+                }
+            }
+        }
+    }
+    if (p.mu && blockIdx.x == 0) { // CTA 0 is the only reader of the old state: it also leaves the new one
+        if (t1 < p.T) {
+            const float r = row(p.T - 1, 0, false);
+            for (int64_t i = (int64_t)threadIdx.x * V; i < W; i += (int64_t)TB * V)
+#pragma unroll
+                for (int c = 0; c < V; c++) before[i + c] = cur[i + c] * r * p.nw[i + c];
+        }
+        for (int64_t i = (int64_t)threadIdx.x * V; i < W; i += (int64_t)TB * V)
+#pragma unroll
+            for (int c = 0; c < V; c++) p.prev[i + c] = before[i + c];
+    }
+}
+
+template <typename E>
+int shift_norm_launch(const shift_norm_args<E> &p) {
+    const size_t smem = (size_t)p.W * 8;
+    const bool vec = p.W % 4 == 0 && (((uintptr_t)p.x | (uintptr_t)p.a | (uintptr_t)p.ls_a | (uintptr_t)p.b | (uintptr_t)p.ls_b | (uintptr_t)p.x_out) & 15) == 0;
+    // tokens per CTA: the row before is computed again once per CTA, so as many as leave two CTAs for every SM
+    int nt = 1;
+    while (!p.rows && nt < 8 && p.T >= (int64_t)nt * 4 * ggb_sm_count()) nt *= 2;
+    const unsigned grid = (unsigned)((p.T + nt - 1) / nt);
+    const bool wide = p.T <= 64 && p.W / (vec ? 4 : 1) >= 512; // a step of few tokens: one pass over the row
+#define SN_LAUNCH(V, TB)                                                                                                        \
+    {                                                                                                                           \
+        auto k = shift_norm_kernel<E, V, TB>;                                                                                   \
+        if (smem > 48 * 1024) GGB_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));         \
+        k<<<grid, TB, smem, ggb_cuda_stream()>>>(p, nt);                                                                        \
+    }
+    if (vec) {
+        if (wide) SN_LAUNCH(4, 512) else SN_LAUNCH(4, 256)
+    } else {
+        if (wide) SN_LAUNCH(1, 512) else SN_LAUNCH(1, 256)
+    }
+#undef SN_LAUNCH
+    GGB_LAUNCH_CHECK();
+    return GGB_OK;
+}
+
+} // namespace
+
+extern "C" {
+
+int ggb_op_xielu_rows(int dt, const float *x, int64_t n, float ap, float an, void *y) {
+    GGB_REQUIRE_INIT();
+    GGB_CHECK_DT(dt);
+    GGB_CHECK_ARG(x && y && n > 0, "xielu_rows: bad arguments");
+    const unsigned blocks = (unsigned)((n + 255) / 256);
+    if (dt == GGB_TYPE_BF16) xielu_rows_kernel<<<blocks, 256, 0, ggb_cuda_stream()>>>(x, n, xielu_args{ap, an}, (__nv_bfloat16 *)y);
+    else xielu_rows_kernel<<<blocks, 256, 0, ggb_cuda_stream()>>>(x, n, xielu_args{ap, an}, (float *)y);
+    GGB_LAUNCH_CHECK();
+    return GGB_OK;
+}
+
+int ggb_op_linear_pair(int dt, const void *w1, int64_t N1, int64_t K1, const void *a1, int64_t lda1, const void *w2, int64_t N2, int64_t K2, const void *a2,
+                       int64_t lda2, int64_t T, float *c1, int64_t ldc1, void *y1, float ap, float an, float *c2, int64_t ldc2) {
+    GGB_REQUIRE_INIT();
+    GGB_CHECK_DT(dt);
+    GGB_CHECK_ARG(w1 && a1 && w2 && a2 && c1 && c2 && T > 0 && N1 > 0 && K1 > 0 && N2 > 0 && K2 > 0 && lda1 >= K1 && lda2 >= K2 && ldc1 >= N1 && ldc2 >= N2 &&
+                      (!y1 || ldc1 == N1),
+                  "linear_pair: bad shape N=%lld / %lld K=%lld / %lld T=%lld", (long long)N1, (long long)N2, (long long)K1, (long long)K2, (long long)T);
+    if (T <= kVecT) { // one launch, the activation as the first product's epilogue
+        const xielu_args xa{ap, an};
+        if (dt == GGB_TYPE_BF16)
+            return linear_pair_launch<__nv_bfloat16>(make_half<__nv_bfloat16>(w1, N1, K1, a1, lda1, c1, y1, ldc1, xa),
+                                                     make_half<__nv_bfloat16>(w2, N2, K2, a2, lda2, c2, nullptr, ldc2, xielu_args{}), T);
+        return linear_pair_launch<float>(make_half<float>(w1, N1, K1, a1, lda1, c1, y1, ldc1, xa),
+                                         make_half<float>(w2, N2, K2, a2, lda2, c2, nullptr, ldc2, xielu_args{}), T);
+    }
+    int rc = ggb_op_linear(dt, w1, N1, K1, a1, lda1, T, c1, ldc1);
+    if (!rc && y1) rc = ggb_op_xielu_rows(dt, c1, T * N1, ap, an, y1);
+    if (!rc) rc = ggb_op_linear(dt, w2, N2, K2, a2, lda2, T, c2, ldc2);
+    return rc;
+}
+
+int ggb_op_shift_norm(int dt, const float *x, const void *table, const int32_t *ids, const float *a, const float *ls_a, const float *b, const float *ls_b,
+                      const float *nw, float eps, const float *mu, float *prev, int64_t W, int64_t T, const int32_t *rows, float *x_out, void *h, void *hs) {
+    GGB_REQUIRE_INIT();
+    GGB_CHECK_DT(dt);
+    GGB_CHECK_ARG((x || (table && ids)) && !(x && table) && W > 0 && T > 0 && (!a || ls_a) && (!b || (a && ls_b)), "shift_norm: an input without its weights");
+    GGB_CHECK_ARG((!mu || (nw && prev && hs && !rows)) && (!h || nw) && (!rows || (h && nw && !x_out)) && (!x_out || x_out != x),
+                  "shift_norm: bad arguments (the renewed rows go to another buffer)");
+    GGB_CHECK_ARG((size_t)W * 8 <= 200 * 1024, "shift_norm: width %lld does not fit shared memory", (long long)W);
+#define SN_CASE(E)                                                                                                                                        \
+    return shift_norm_launch<E>(shift_norm_args<E>{x, (const E *)table, ids, a, ls_a, b, ls_b, nw, mu, eps, W, T, rows, prev, x_out, (E *)h, (E *)hs});
+    if (dt == GGB_TYPE_BF16) SN_CASE(__nv_bfloat16)
+    SN_CASE(float)
+#undef SN_CASE
 }
 
 } // extern "C"

@@ -35,6 +35,9 @@ int ggb_norm_add_norm_launch(int dt, const float *a, const float *bias, const in
                              int64_t E, int64_t T, float *x, const float *wy, void *y);
 
 #ifdef __CUDACC__
+__device__ __forceinline__ float gelu_tanh_f32(float z) {
+    return 0.5f * z * (1.0f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
+}
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
 template <typename E> __device__ __forceinline__ E from_f32(float v);

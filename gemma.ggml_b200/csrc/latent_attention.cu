@@ -21,15 +21,36 @@ namespace {
 
 __device__ __forceinline__ int64_t cache_row(const int32_t *table, int B, int64_t j) { return (int64_t)table[j / B] * B + j % B; }
 
+// rotated pair m of a vector whose first `dims` numbers turn: the neighbours (2m, 2m + 1), or with `halves` (m, m + dims / 2)
+// for the turned pairs and the neighbours behind them for the rest
+__device__ __forceinline__ void rot_pair(int m, int dims, int halves, int *i0, int *i1) {
+    const bool half = halves && 2 * m < dims;
+    *i0 = half ? m : 2 * m;
+    *i1 = half ? m + dims / 2 : 2 * m + 1;
+}
+
 // ---- c = rms(d[:R]) * nw, kr = rot(d[R:]) into the cache rows of the step's tokens.  One CTA per token.
-// cs: [n_pos][dims / 2][2] (cos, sin) with the rotation's magnitude factor already applied.
+// cs: [n_pos][dims / 2][2] (cos, sin) with the rotation's magnitude factor already applied.  blockIdx.y 1: the query latent
+// of the same token instead, cq = rms(dq) * qnw.
 template <typename E>
 __global__ void __launch_bounds__(128) latent_kv_store_kernel(const float *__restrict__ d, int64_t ldd, int R, int Dr, int dims,
                                                               const float *__restrict__ nw, float eps, const float *__restrict__ cs,
                                                               const int32_t *__restrict__ pos0, const int32_t *__restrict__ table,
-                                                              int B, E *__restrict__ cache, int64_t ldk) {
+                                                              int B, E *__restrict__ cache, int64_t ldk, int halves,
+                                                              const float *__restrict__ dq, int Rq, const float *__restrict__ qnw, E *__restrict__ cq) {
     __shared__ float red[4];
     const int t = blockIdx.x, tid = threadIdx.x;
+    if (blockIdx.y == 1) {
+        const float *qr = dq + (int64_t)t * ldd;
+        float ss = 0.f;
+        for (int i = tid; i < Rq; i += 128) ss = fmaf(qr[i], qr[i], ss);
+        ss = warp_sum_f32(ss);
+        if ((tid & 31) == 0) red[tid >> 5] = ss;
+        __syncthreads();
+        const float r = 1.0f / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)Rq + eps);
+        for (int i = tid; i < Rq; i += 128) cq[(int64_t)t * Rq + i] = from_f32<E>(qr[i] * r * qnw[i]);
+        return;
+    }
     const float *dr = d + (int64_t)t * ldd;
     const int64_t p = (int64_t)*pos0 + t;
     E *row = cache + cache_row(table, B, p) * ldk;
@@ -42,7 +63,8 @@ __global__ void __launch_bounds__(128) latent_kv_store_kernel(const float *__res
     for (int i = tid; i < R; i += 128) row[i] = from_f32<E>(dr[i] * r * nw[i]);
     const float *tab = cs + p * dims; // dims / 2 pairs of (cos, sin)
     for (int i = tid; i < Dr / 2 + (Dr & 1); i += 128) {
-        const int i0 = 2 * i, i1 = 2 * i + 1;
+        int i0, i1;
+        rot_pair(i, dims, halves, &i0, &i1);
         if (i1 < dims) {
             const float u = dr[R + i0], v = dr[R + i1], c = tab[2 * i], s = tab[2 * i + 1];
             row[R + i0] = from_f32<E>(u * c - v * s);
@@ -61,7 +83,8 @@ constexpr int kAbsT = 8;
 template <typename E>
 __global__ void __launch_bounds__(256) latent_q_absorb_kernel(const float *__restrict__ q, int64_t ldq, int64_t T, int H, int D, int Dr,
                                                               int dims, const float *__restrict__ cs, const int32_t *__restrict__ pos0,
-                                                              const E *__restrict__ w_uk, int R, float scale, float *__restrict__ qa) {
+                                                              const E *__restrict__ w_uk, int R, float scale, float *__restrict__ qa,
+                                                              int halves) {
     extern __shared__ float qs[]; // [kAbsT][D], then [4][kAbsT][64] partial sums
     float *ps = qs + kAbsT * D;
     const int h = blockIdx.y, tid = threadIdx.x, rl = tid & 63, dg = tid >> 6;
@@ -106,7 +129,8 @@ __global__ void __launch_bounds__(256) latent_q_absorb_kernel(const float *__res
         const int64_t t = t0 + tt, p = (int64_t)*pos0 + t;
         const float *src = q + t * ldq + (int64_t)h * (D + Dr) + D;
         float *dst = qa + (t * H + h) * QK + R;
-        const int i0 = 2 * pi, i1 = i0 + 1;
+        int i0, i1;
+        rot_pair(pi, dims, halves, &i0, &i1);
         if (i1 < dims) {
             const float u = src[i0], v = src[i1], c = cs[p * dims + 2 * pi], sn = cs[p * dims + 2 * pi + 1];
             dst[i0] = (u * c - v * sn) * scale;
@@ -418,6 +442,52 @@ __global__ void latent_gather_kernel(const E *__restrict__ cache, int64_t ldk, c
     for (int i = threadIdx.x; i < R; i += blockDim.x) out[(int64_t)blockIdx.x * R + i] = row[i];
 }
 
+// materialised keys with a rotated part: kvf rows [k (H D) | v (H Dv)] and the cache's shared rotated part become rows
+// [k (H (D + Dr)) | v (H Dv)], the rotated part repeated behind every head's own
+template <typename E>
+__global__ void __launch_bounds__(256) latent_pack_kernel(const float *__restrict__ kvf, const E *__restrict__ cache, int64_t ldk, const int32_t *__restrict__ table,
+                                                          int B, int64_t first, int R, int H, int D, int Dr, int Dv, E *__restrict__ kv, int64_t ld_kv) {
+    const int64_t n = blockIdx.x;
+    const E *kr = cache + cache_row(table, B, first + n) * ldk + R;
+    const float *src = kvf + n * (int64_t)H * (D + Dv);
+    const int nk = H * (D + Dr), nv = H * Dv, DD = D + Dr;
+    for (int i = threadIdx.x; i < nk + nv; i += blockDim.x) {
+        E x;
+        if (i < nk) {
+            const int h = i / DD, d = i - h * DD;
+            x = d < D ? from_f32<E>(src[h * D + d]) : kr[d - D];
+        } else {
+            x = from_f32<E>(src[H * D + i - nk]);
+        }
+        kv[n * ld_kv + i] = x;
+    }
+}
+
+// q rows [H][D + Dr] times scale, the last Dr of every head turned: what a materialised key is scored against
+__global__ void __launch_bounds__(256) latent_q_rotate_kernel(const float *__restrict__ q, int64_t ldq, int H, int D, int Dr, int dims, int halves,
+                                                              const float *__restrict__ cs, const int32_t *__restrict__ pos0, float scale,
+                                                              float *__restrict__ out) {
+    const int64_t t = blockIdx.x, p = (int64_t)*pos0 + t;
+    const int DD = D + Dr, half = Dr / 2 + (Dr & 1);
+    for (int i = threadIdx.x; i < H * DD; i += blockDim.x)
+        if (i % DD < D) out[t * H * DD + i] = q[t * ldq + i] * scale;
+    for (int i = threadIdx.x; i < H * half; i += blockDim.x) {
+        const int h = i / half, pi = i - h * half;
+        const float *src = q + t * ldq + (int64_t)h * DD + D;
+        float *dst = out + (t * H + h) * DD + D;
+        int i0, i1;
+        rot_pair(pi, dims, halves, &i0, &i1);
+        if (i1 < dims) {
+            const float u = src[i0], v = src[i1], c = cs[p * dims + 2 * pi], sn = cs[p * dims + 2 * pi + 1];
+            dst[i0] = (u * c - v * sn) * scale;
+            dst[i1] = (v * c + u * sn) * scale;
+        } else {
+            dst[i0] = src[i0] * scale;
+            if (i1 < Dr) dst[i1] = src[i1] * scale;
+        }
+    }
+}
+
 template <typename E>
 __global__ void cvt_rows_kernel(const float *__restrict__ x, int64_t n, E *__restrict__ y) {
     const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -476,26 +546,40 @@ extern "C" {
 
 int64_t ggb_latent_cache_ld(int R, int Dr) { return ((int64_t)R + Dr + 7) / 8 * 8; }
 
-int ggb_op_latent_kv_store(int dt, const float *d, int64_t ldd, int64_t T, int R, int Dr, int rot_dims, const float *norm_w, float eps,
-                           const float *cos_sin, const int32_t *pos0, const int32_t *block_table, int block_size, void *cache) {
+static int latent_kv_store_launch(int dt, const float *d, int64_t ldd, int64_t T, int R, int Dr, int rot_dims, int halves, const float *norm_w,
+                                  const float *dq, int Rq, const float *q_norm_w, void *cq, float eps, const float *cos_sin, const int32_t *pos0,
+                                  const int32_t *block_table, int block_size, void *cache) {
     GGB_REQUIRE_INIT();
     GGB_CHECK_DT(dt);
     GGB_CHECK_ARG(d && norm_w && (cos_sin || !rot_dims) && pos0 && block_table && cache && T > 0 && R > 0 && Dr >= 0 && block_size > 0 &&
-                      rot_dims >= 0 && rot_dims <= Dr && rot_dims % 2 == 0,
+                      rot_dims >= 0 && rot_dims <= Dr && rot_dims % 2 == 0 && (!dq || (Rq > 0 && q_norm_w && cq)),
                   "latent_kv_store: bad arguments");
     const int64_t ldk = ggb_latent_cache_ld(R, Dr);
+    const dim3 grid((unsigned)T, dq ? 2 : 1);
     if (dt == GGB_TYPE_BF16)
-        latent_kv_store_kernel<<<(unsigned)T, 128, 0, ggb_cuda_stream()>>>(d, ldd, R, Dr, rot_dims, norm_w, eps, cos_sin, pos0, block_table,
-                                                                           block_size, (__nv_bfloat16 *)cache, ldk);
+        latent_kv_store_kernel<<<grid, 128, 0, ggb_cuda_stream()>>>(d, ldd, R, Dr, rot_dims, norm_w, eps, cos_sin, pos0, block_table, block_size,
+                                                                    (__nv_bfloat16 *)cache, ldk, halves, dq, Rq, q_norm_w, (__nv_bfloat16 *)cq);
     else
-        latent_kv_store_kernel<<<(unsigned)T, 128, 0, ggb_cuda_stream()>>>(d, ldd, R, Dr, rot_dims, norm_w, eps, cos_sin, pos0, block_table,
-                                                                           block_size, (float *)cache, ldk);
+        latent_kv_store_kernel<<<grid, 128, 0, ggb_cuda_stream()>>>(d, ldd, R, Dr, rot_dims, norm_w, eps, cos_sin, pos0, block_table, block_size,
+                                                                    (float *)cache, ldk, halves, dq, Rq, q_norm_w, (float *)cq);
     GGB_LAUNCH_CHECK();
     return GGB_OK;
 }
 
-int ggb_op_latent_q_absorb(int dt, const float *q, int64_t ldq, int64_t T, int H, int D, int Dr, int rot_dims, const float *cos_sin,
-                           const int32_t *pos0, const void *w_uk, int R, float scale, float *qa) {
+int ggb_op_latent_kv_store(int dt, const float *d, int64_t ldd, int64_t T, int R, int Dr, int rot_dims, const float *norm_w, float eps,
+                           const float *cos_sin, const int32_t *pos0, const int32_t *block_table, int block_size, void *cache) {
+    return latent_kv_store_launch(dt, d, ldd, T, R, Dr, rot_dims, 0, norm_w, nullptr, 0, nullptr, nullptr, eps, cos_sin, pos0, block_table, block_size, cache);
+}
+
+int ggb_op_latent_prep(int dt, const float *dq, int Rq, const float *q_norm_w, void *cq, const float *dkv, int64_t ld, int64_t T, int R, int Dr,
+                       int rot_dims, int rot_halves, const float *kv_norm_w, float eps, const float *cos_sin, const int32_t *pos0,
+                       const int32_t *block_table, int block_size, void *cache) {
+    return latent_kv_store_launch(dt, dkv, ld, T, R, Dr, rot_dims, rot_halves, kv_norm_w, dq, Rq, q_norm_w, cq, eps, cos_sin, pos0, block_table, block_size,
+                                  cache);
+}
+
+static int latent_q_absorb_launch(int dt, const float *q, int64_t ldq, int64_t T, int H, int D, int Dr, int rot_dims, int halves, const float *cos_sin,
+                                  const int32_t *pos0, const void *w_uk, int R, float scale, float *qa) {
     GGB_REQUIRE_INIT();
     GGB_CHECK_DT(dt);
     GGB_CHECK_ARG(q && (cos_sin || !rot_dims) && pos0 && w_uk && qa && T > 0 && H > 0 && D > 0 && R > 0 && rot_dims <= Dr && rot_dims % 2 == 0,
@@ -505,10 +589,51 @@ int ggb_op_latent_q_absorb(int dt, const float *q, int64_t ldq, int64_t T, int H
     GGB_CHECK_ARG(smem <= 48 * 1024, "latent_q_absorb: head dimension %d too large", D);
     if (dt == GGB_TYPE_BF16)
         latent_q_absorb_kernel<<<grid, 256, smem, ggb_cuda_stream()>>>(q, ldq, T, H, D, Dr, rot_dims, cos_sin, pos0,
-                                                                       (const __nv_bfloat16 *)w_uk, R, scale, qa);
+                                                                       (const __nv_bfloat16 *)w_uk, R, scale, qa, halves);
     else
         latent_q_absorb_kernel<<<grid, 256, smem, ggb_cuda_stream()>>>(q, ldq, T, H, D, Dr, rot_dims, cos_sin, pos0, (const float *)w_uk, R,
-                                                                       scale, qa);
+                                                                       scale, qa, halves);
+    GGB_LAUNCH_CHECK();
+    return GGB_OK;
+}
+
+int ggb_op_latent_q_absorb(int dt, const float *q, int64_t ldq, int64_t T, int H, int D, int Dr, int rot_dims, const float *cos_sin,
+                           const int32_t *pos0, const void *w_uk, int R, float scale, float *qa) {
+    return latent_q_absorb_launch(dt, q, ldq, T, H, D, Dr, rot_dims, 0, cos_sin, pos0, w_uk, R, scale, qa);
+}
+
+int ggb_op_latent_q_absorb_halves(int dt, const float *q, int64_t ldq, int64_t T, int H, int D, int Dr, int rot_dims, const float *cos_sin,
+                                  const int32_t *pos0, const void *w_uk, int R, float scale, float *qa) {
+    return latent_q_absorb_launch(dt, q, ldq, T, H, D, Dr, rot_dims, 1, cos_sin, pos0, w_uk, R, scale, qa);
+}
+
+int ggb_op_latent_q_rotate(const float *q, int64_t ldq, int64_t T, int H, int D, int Dr, int rot_dims, int rot_halves, const float *cos_sin,
+                           const int32_t *pos0, float scale, float *out) {
+    GGB_REQUIRE_INIT();
+    GGB_CHECK_ARG(q && out && pos0 && (cos_sin || !rot_dims) && T > 0 && H > 0 && D >= 0 && Dr >= 0 && rot_dims <= Dr && rot_dims % 2 == 0 &&
+                      ldq >= (int64_t)H * (D + Dr),
+                  "latent_q_rotate: bad arguments");
+    latent_q_rotate_kernel<<<(unsigned)T, 256, 0, ggb_cuda_stream()>>>(q, ldq, H, D, Dr, rot_dims, rot_halves, cos_sin, pos0, scale, out);
+    GGB_LAUNCH_CHECK();
+    return GGB_OK;
+}
+
+int ggb_op_latent_expand_rot(int dt, const void *cache, const int32_t *block_table, int block_size, int64_t first, int64_t n, int R, int H, int D,
+                             int Dr, int Dv, const void *w_ukv, void *c_rows, float *kv_f32, void *kv, int64_t ld_kv) {
+    GGB_REQUIRE_INIT();
+    GGB_CHECK_DT(dt);
+    GGB_CHECK_ARG(cache && block_table && w_ukv && c_rows && kv && kv_f32 && block_size > 0 && first >= 0 && n > 0 && R > 0 && H > 0 && D > 0 && Dr >= 0 &&
+                      Dv > 0 && ld_kv >= (int64_t)H * (D + Dr + Dv),
+                  "latent_expand_rot: bad arguments");
+    const int64_t ldk = ggb_latent_cache_ld(R, Dr), N = (int64_t)H * (D + Dv);
+#define LE_CASE(E)                                                                                                                                        \
+    latent_gather_kernel<<<(unsigned)n, 128, 0, ggb_cuda_stream()>>>((const E *)cache, ldk, block_table, block_size, first, R, (E *)c_rows);               \
+    GGB_LAUNCH_CHECK();                                                                                                                                   \
+    const int rc = ggb_op_linear(dt, w_ukv, N, R, c_rows, R, n, kv_f32, N);                                                                                \
+    if (rc) return rc;                                                                                                                                    \
+    latent_pack_kernel<<<(unsigned)n, 256, 0, ggb_cuda_stream()>>>(kv_f32, (const E *)cache, ldk, block_table, block_size, first, R, H, D, Dr, Dv, (E *)kv, ld_kv);
+    if (dt == GGB_TYPE_BF16) { LE_CASE(__nv_bfloat16) } else { LE_CASE(float) }
+#undef LE_CASE
     GGB_LAUNCH_CHECK();
     return GGB_OK;
 }

@@ -12,6 +12,7 @@
 #include "begupel_model.h"
 #include "ditalorn_model.h"
 #include "kibilix_model.h"
+#include "tezesun_model.h"
 #include "safolorn_model.h"
 #include "tensor_dump.h"
 
@@ -256,6 +257,23 @@ int kb_config_probe(const char *text, int64_t *out) {
     for (const auto &l : c.layers) moe += l.ff_kind == 2;
     out[0] = (int64_t)c.layers.size(); out[1] = (int64_t)c.runs.size(); out[2] = attn; out[3] = delta; out[4] = moe; out[5] = c.vocab;
     out[6] = c.width; out[7] = c.streams;
+    return 0;
+}
+// host only: parses a Tezesun configuration text; out[9] = {layers, attention layers, latent layers, rglru layers, layers with a
+// feed-forward, vocab, width, widest window (0: some layer sees everything), kept first tokens}; -1 and gm_last_error() when it is
+// refused
+int tz_config_probe(const char *text, int64_t *out) {
+    json_value j;
+    tz_config c;
+    if (!json_parser(text, strlen(text)).parse(&j, &g_capi_err)) return -1;
+    if (tz_parse_config(j, nullptr, &c, &g_capi_err)) return -1;
+    int64_t n[3] = {0, 0, 0}, ff = 0;
+    for (const auto &l : c.layers) {
+        n[l.type]++;
+        ff += l.ff > 0;
+    }
+    out[0] = (int64_t)c.layers.size(); out[1] = n[0]; out[2] = n[1]; out[3] = n[2]; out[4] = ff; out[5] = c.vocab; out[6] = c.width;
+    tz_lookback(c, &out[7], &out[8]);
     return 0;
 }
 // host only: a tensor of a .safetensors file: returns its number of dimensions (shape[0 .. 8) filled, *nbytes, dtype text),

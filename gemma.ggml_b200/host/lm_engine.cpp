@@ -99,7 +99,7 @@ int lm_engine::run_entry(const lm_entry &e, std::vector<float> *logits, int32_t 
     }
     s.len += n;
     // rows no later token can see: their pages serve other sequences from now on
-    if (model_->cache_lookback() > 0) cache_.trim(s.slot, s.len - model_->cache_lookback() + 1);
+    if (model_->cache_lookback() > 0) cache_.trim(s.slot, s.len - model_->cache_lookback() + 1, model_->cache_keep_first());
     return 0;
 }
 

@@ -37,6 +37,8 @@ class lm_model {
     // how many positions back the farthest-looking caching layer reads (0: unbounded): the engine gives back the pages
     // before that while the sequence lives
     virtual int64_t cache_lookback() const { return 0; }
+    // with a lookback: how many first positions of a sequence stay visible all the same (their pages are kept)
+    virtual int64_t cache_keep_first() const { return 0; }
     virtual int max_live_sequences() const { return 0; } // 0: as many as the engine has slots
     virtual int max_portion() const = 0; // most tokens one forward call takes; the engine cuts longer portions
     // runs the portion from the state earlier portions left in the cache; the logits of rows want[0 .. n_want) of the

@@ -47,7 +47,7 @@ int paged_cache::open_seq() {
         if (!seqs_[i].open) {
             seqs_[i].open = true;
             seqs_[i].pages.clear();
-            seqs_[i].trimmed = 0;
+            seqs_[i].trimmed = seqs_[i].given_back = 0;
             if (state_ && ggb_buffer_memset(state((int)i), 0, (size_t)state_elems_ * 4)) return -1; // stream-ordered: before the first step
             return (int)i;
         }
@@ -81,22 +81,24 @@ void paged_cache::close_seq(int slot) {
     for (size_t i = s.pages.size(); i-- > 0;)
         if (s.pages[i] >= 0) free_.push_back(s.pages[i]); // the first page is reused first
     s.pages.clear();
-    s.trimmed = 0;
+    s.trimmed = s.given_back = 0;
     s.open = false;
 }
 
-void paged_cache::trim(int slot, int64_t first_needed) {
+void paged_cache::trim(int slot, int64_t first_needed, int64_t keep_first) {
     seq &s = seqs_[(size_t)slot];
     if (first_needed <= 0) return;
     const size_t keep_from = std::min((size_t)(first_needed / page_), s.pages.size());
-    for (size_t i = s.trimmed; i < keep_from; i++) {
+    const size_t kept = (size_t)((std::max<int64_t>(keep_first, 0) + page_ - 1) / page_);
+    for (size_t i = std::max(s.trimmed, kept); i < keep_from; i++) {
         free_.push_back(s.pages[i]);
         s.pages[i] = -1;
+        s.given_back++;
     }
     if (keep_from > s.trimmed) s.trimmed = keep_from;
 }
 
 int paged_cache::live_pages(int slot) const {
     const seq &s = seqs_[(size_t)slot];
-    return (int)(s.pages.size() - s.trimmed);
+    return (int)(s.pages.size() - s.given_back);
 }

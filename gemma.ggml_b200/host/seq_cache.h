@@ -6,7 +6,8 @@
 // Beside the rows a sequence may carry a block of fixed size (fp32 numbers: recurrent state, tails of convolutions, the
 // previous token): one per slot, zeroed when the slot is opened, so a slot that is used again starts clean.  Models
 // whose caching layers all look back a bounded number of positions let the engine trim: pages that lie wholly before
-// the earliest position any later token can see go back to the free list while the sequence lives.
+// the earliest position any later token can see go back to the free list while the sequence lives (except the first ones of
+// a sequence, when the model keeps those visible for good).
 #pragma once
 
 #include <cstdint>
@@ -22,8 +23,9 @@ class paged_cache {
     int open_seq();                         // slot (its state block zeroed), or -1 when all slots are taken
     int reserve(int slot, int64_t n_tokens); // pages for n_tokens positions (0 ok, -1: out of pages); table uploaded
     void close_seq(int slot);
-    // gives back the pages that hold only positions < first_needed; their table entries stay but are never read again
-    void trim(int slot, int64_t first_needed);
+    // gives back the pages that hold only positions in [keep_first, first_needed); their table entries stay but are never
+    // read again
+    void trim(int slot, int64_t first_needed, int64_t keep_first = 0);
     float *state(int slot) const { return state_ ? state_ + (size_t)slot * (size_t)state_elems_ : nullptr; }
     int64_t state_elems() const { return state_elems_; }
     int live_pages(int slot) const;
@@ -41,7 +43,8 @@ class paged_cache {
     struct seq {
         bool open = false;
         std::vector<int32_t> pages; // -1: trimmed
-        size_t trimmed = 0;         // pages [0, trimmed) are given back
+        size_t trimmed = 0;         // pages before this one were looked at: all but the kept first ones are given back
+        size_t given_back = 0;
     };
     int dt_ = 0, page_ = 0, n_pages_ = 0;
     std::vector<void *> layers_;

@@ -321,6 +321,44 @@ int ggb_op_linear_relu2(int dt, const void *w, int64_t N, int64_t K, const void 
 /* y (dt, dense [T][F]) = act(x), x fp32 rows of stride ldx; act 0: as it is, 1: relu(x)^2 */
 int ggb_op_act_rows(int dt, const float *x, int64_t ldx, int64_t T, int64_t F, int act, void *y);
 
+/* Layers whose two sublayers read one normed input side by side.  One pass between two such layers: x' = x + (a * ls_a +
+ * b * ls_b) per channel (a, then b, may be NULL) -> x_out (fp32, another buffer than x, may be NULL); h = x' / sqrt(mean(x'^2) +
+ * eps) * nw in dt (nw NULL: none; h may be NULL); with mu the token shift hs = h + (h_before - h) * mu in dt, h_before the row of
+ * the token before, in fp32: for the portion's first token prev (fp32 [W], the sequence's state, zeros at its start), which is
+ * replaced by the portion's last row.  table / ids (with x NULL): the residual starts as the tokens' embedding rows.
+ * rows (device int32): only the tokens rows[0 .. T), h only (no shift, no x_out). */
+int ggb_op_shift_norm(int dt, const float *x, const void *table, const int32_t *ids, const float *a, const float *ls_a, const float *b, const float *ls_b,
+                      const float *nw, float eps, const float *mu, float *prev, int64_t W, int64_t T, const int32_t *rows, float *x_out, void *h, void *hs);
+/* two products of different inputs: c1 = a1 w1^T and c2 = a2 w2^T (fp32).  With y1 (dt, [T][N1], ldc1 == N1) the first one leaves
+ * as xielu (below) and c1 is scratch.  T <= 8: one launch, the activation as its epilogue; else as ggb_op_linear. */
+int ggb_op_linear_pair(int dt, const void *w1, int64_t N1, int64_t K1, const void *a1, int64_t lda1, const void *w2, int64_t N2, int64_t K2, const void *a2,
+                       int64_t lda2, int64_t T, float *c1, int64_t ldc1, void *y1, float ap, float an, float *c2, int64_t ldc2);
+/* y (dt) = xielu(x): z > 0: ap z^2 + z / 2; z <= 0: an (exp(z) - 1 - z) + z / 2 */
+int ggb_op_xielu_rows(int dt, const float *x, int64_t n, float ap, float an, void *y);
+
+/* ------------------------------------------------------------------ gated diagonal linear recurrence (csrc/rglru.cu)
+ * C = nb * d channels.  u_t = conv_b + sum_j conv_w[c][j] (x + xb)_(t - taps + 1 + j) (the last tap weighs the current token, taps
+ * <= 8); per block b of d channels the gates r | i = sigmoid(w_ri[b] u[b] + b_ri[b]) with w_ri [nb][2d][d] in dt (the rows of r, then
+ * of i) and b_ri [nb][2d]; log a = rate[c] r; S <- a S + sqrt(1 - a^2) i u; out (dt, [T][C]) = S * gelu_tanh(y + yb).  x, y: fp32
+ * rows of stride ld.  State (fp32): S [C] and the convolution's last inputs, a ring hist [ggb_rglru_history_rows(taps)][C]
+ * indexed by position (*pos0 + t, read on the device).  A portion continues from what the one before left.
+ *
+ * step: T <= 8 (ggb_rglru_step_form), one launch.  Portions: conv -> gates -> scan; conv also writes u as three bf16 numbers that
+ * sum to it (split [nb][T][3d], offsets [nb + 1]; ggb_rglru_split_fits), which the gates multiply on the tensor cores by
+ * w_ri3 [nb][2d][3d] (every row of w_ri three times); without split the gates run in fp32.  z [nb][T][2d] fp32. */
+int ggb_rglru_history_rows(int taps);
+int ggb_rglru_step_form(int64_t T, int d);
+int ggb_rglru_split_fits(int dt, int64_t T, int d);
+int ggb_op_rglru_step(int dt, const float *x, const float *y, int64_t ld, int64_t T, int nb, int d, const float *conv_w, const float *conv_b, int taps,
+                      const float *xb, const float *yb, const void *w_ri, const float *b_ri, const float *rate, const int32_t *pos0, float *hist,
+                      float *state, void *out);
+int ggb_op_rglru_conv(const float *x, int64_t ld, int64_t T, int nb, int d, const float *conv_w, const float *conv_b, int taps, const float *xb,
+                      const int32_t *pos0, float *hist, float *u, void *split, int32_t *offsets);
+int ggb_op_rglru_gates(int dt, const float *u, const void *split, const int32_t *offsets, int64_t T, int nb, int d, const void *w_ri, const void *w_ri3,
+                       float *z);
+int ggb_op_rglru_scan(int dt, const float *z, const float *u, const float *y, int64_t ld, int64_t T, int nb, int d, const float *yb, const float *b_ri,
+                      const float *rate, float *state, void *out);
+
 /* ------------------------------------------------------------------ recurrent mixers (csrc/recurrent.cu)
  * State that a sequence carries from token to token (fp32, one block per sequence, handed in by the caller): tails of
  * causal convolutions and the matrices S [heads][D][Dv] of linear-attention recurrences.
@@ -394,6 +432,21 @@ int ggb_op_masked_attn(int dt, const float *q, const void *cache, const int32_t 
                        int H, int G, int D, int Dv, int64_t window, int chunked, float softcap, const float *cos_sin_v, void *out,
                        float *scratch);
 
+/* a window that keeps the first positions visible: the query at position i sees j <= i with i - j < window or j < keep_first */
+int ggb_op_masked_attn_keep(int dt, const float *q, const void *cache, const int32_t *block_table, int block_size, const int32_t *pos0, int64_t T,
+                            int H, int G, int D, int Dv, int64_t window, int64_t keep_first, float softcap, void *out, float *scratch);
+/* Differential attention: every head has two query / key maps over the same values.  q [T][H][2][D], k [T][G][2][D], v
+ * [T][G][Dv] raw projections; cache row [k (G * 2 * D) | v (G * Dv)], ggb_window_cache_ld(G, 2 * D, Dv) numbers apart; q_out
+ * [T][H][2][D].  Each map is a soft-max attention of its own (window, keep_first, softcap as above); with a1, a2 their outputs
+ * o = a1 - lambda a2, out (dt, [T][H * Dv]) = o / sqrt(mean over the head (o^2) + eps) * out_scale * sigmoid(gate) (gate fp32 rows
+ * of stride ldg, a number per output; NULL: no gate).  scratch: ggb_window_attn_scratch_bytes(2 * H). */
+int ggb_op_diff_qkv_store(int dt, const float *q, const float *k, const float *v, int64_t ld, int64_t T, int H, int G, int D, int Dv, int rot_dims,
+                          int rot_halves, const float *cos_sin_k, float scale, const int32_t *pos0, const int32_t *block_table, int block_size,
+                          void *cache, float *q_out);
+int ggb_op_diff_attn(int dt, const float *q, const void *cache, const int32_t *block_table, int block_size, const int32_t *pos0, int64_t T, int H,
+                     int G, int D, int Dv, int64_t window, int64_t keep_first, float softcap, float lambda, float out_scale, float eps,
+                     const float *gate, int64_t ldg, void *out, float *scratch);
+
 /* ------------------------------------------------------------------ sigmoid attention (csrc/sigmoid_attention.cu)
  * Grouped-query attention with unnormalised weights over the same paged rows [k (G * D) | v (G * Dv)] (ggb_window_cache_ld):
  * the weight of key j for the query at position i is sigmoid(q . k - r1[h] ln(1 + r2[h] (i - j)) + pb[h]), the output
@@ -444,6 +497,20 @@ int ggb_op_latent_attn_window(int dt, const float *qa, const void *cache, const 
  * and positions counted from `first`.  kv_f32 ([n][ld_kv] fp32) is scratch for the bf16 type. */
 int ggb_op_latent_expand(int dt, const void *cache, const int32_t *block_table, int block_size, int64_t first, int64_t n, int R, int Dr,
                          const void *w_ukv, int64_t N, void *c_rows, float *kv_f32, void *kv, int64_t ld_kv);
+/* Rotary pairs in the halves layout (m, m + rot_dims / 2), and both latents of a layer in one launch: cq (dt, [T][Rq]) =
+ * rms(dq) * q_norm_w beside what ggb_op_latent_kv_store does with dkv (dq NULL: that alone); dq and dkv rows of stride ld */
+int ggb_op_latent_prep(int dt, const float *dq, int Rq, const float *q_norm_w, void *cq, const float *dkv, int64_t ld, int64_t T, int R, int Dr,
+                       int rot_dims, int rot_halves, const float *kv_norm_w, float eps, const float *cos_sin, const int32_t *pos0,
+                       const int32_t *block_table, int block_size, void *cache);
+int ggb_op_latent_q_absorb_halves(int dt, const float *q, int64_t ldq, int64_t T, int H, int D, int Dr, int rot_dims, const float *cos_sin,
+                                  const int32_t *pos0, const void *w_uk, int R, float scale, float *qa);
+/* the materialised form with a rotated part: kv rows [k (H (D + Dr)) | v (H Dv)], every head's key followed by the shared
+ * rotated part; kv_f32 ([n][H (D + Dv)] fp32) is scratch in both types.  q_rotate: out [T][H][D + Dr] = scale * (q with the last Dr
+ * numbers of every head turned), what those keys are scored against. */
+int ggb_op_latent_expand_rot(int dt, const void *cache, const int32_t *block_table, int block_size, int64_t first, int64_t n, int R, int H, int D,
+                             int Dr, int Dv, const void *w_ukv, void *c_rows, float *kv_f32, void *kv, int64_t ld_kv);
+int ggb_op_latent_q_rotate(const float *q, int64_t ldq, int64_t T, int H, int D, int Dr, int rot_dims, int rot_halves, const float *cos_sin,
+                           const int32_t *pos0, float scale, float *out);
 /* x (dt, [T][H * Dv], in place): head h of token t times sigmoid(gate[t * ldg + h]) */
 int ggb_op_head_gate(int dt, void *x, int64_t T, int H, int Dv, const float *gate, int64_t ldg);
 /* the merge without a sink (sink NULL: ordinary soft-max over the keys) and / or with an output gate: head h of token t
