@@ -841,6 +841,33 @@ def _begupel_record(G, peaks, dims, T, ctx, n_dec):
     return rec
 
 
+def _safolorn_record(G, peaks, W, nl, H, D, ff, V, T, ctx, n_dec):
+    """Safolorn at equal size: latent attention with heads of the same size, dense feed-forward everywhere"""
+    R = 512 if W >= 2048 else 256
+    mx = {"heads": H, "dim": D, "rot_dim": 64, "vdim": D, "kv_rank": R, "scale": (D + 64) ** -0.5,
+          "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    scfg = {"architecture": "Safolorn", "vocab": V, "width": W, "norm": {"eps": 1e-5},
+            "layers": [{"type": "latent_attention", "mixer": mx, "mlp": {"kind": "dense", "ff": ff, "limit": 7.0}} for _ in range(nl)]}
+    seng = G.Engine(config=scfg, seed=7, dtype="bfloat16", max_tokens=ctx + n_dec + 64, page_size=64, max_portion=1024)
+    spf, spf_ops, sdec, sdc_ops, skernels, _ = _engine_times(G, seng, V, T, ctx, n_dec, BG_OPS)
+    s_params = nl * (W * (H * (D + 64) + R + 64) + W * H * D + 3.0 * ff * W)
+    s_flops, s_bytes = 2.0 * T * s_params + 2.0 * V * W, 2.0 * (s_params + V * W)
+    s_attn = 2.0 * nl * H * (2 * R + 64) * T * (T + 1) / 2
+    s_cache = 2.0 * nl * ctx * (R + 64)
+    rec = {
+        "config": {"kv_rank": R, "rot_dim": 64, "weight_bytes": seng.stats()["weight_bytes"]},
+        "prefill": {"tokens_per_s": T / spf, "ms": 1e3 * spf, "op_ms": spf_ops, "linear_tflops": s_flops / (spf_ops["op_linear"] / 1e3) / 1e12,
+                    "linear_frac_of_tensor_peak": s_flops / (spf_ops["op_linear"] / 1e3) / 1e12 / peaks["bf16_tflops_sustained"],
+                    "attn_tflops_cuda_cores": s_attn / (spf_ops["op_attn"] / 1e3) / 1e12},
+        "decode": {"tokens_per_s": 1.0 / sdec, "us_per_token": 1e6 * sdec, "kernels_per_token": skernels, "op_us": {k: 1e3 * v for k, v in sdc_ops.items()},
+                   "linear_gbs": s_bytes / (sdc_ops["op_linear"] / 1e3) / 1e9, "linear_frac_of_hbm_peak": s_bytes / (sdc_ops["op_linear"] / 1e3) / 1e9 / peaks["hbm_gbs"],
+                   "attn_gbs": s_cache / (sdc_ops["op_attn"] / 1e3) / 1e9,
+                   "token_frac_of_hbm_roofline": ((s_bytes + s_cache) / (peaks["hbm_gbs"] * 1e9)) / sdec},
+    }
+    seng.close()
+    return rec
+
+
 def run_begupel(args):
     """--arch begupel: prefill and decode throughput of the Begupel design (random bf16 weights) at layer sizes of real
     models, through the serving engine (host call: H2D token ids, operator launches / graph replay, D2H result), with
@@ -859,29 +886,8 @@ def run_begupel(args):
     for size in args.sizes.split(","):
         W, nl, H, Gk, D, win, Hr, Gr, Hl, ff, V = BEGUPEL_SIZES[size]
         rec = _begupel_record(G, peaks, BEGUPEL_SIZES[size], T, ctx, n_dec)
-        if not args.no_sub_records:  # Safolorn at equal size: latent attention with heads of the same size, dense feed-forward everywhere
-            R = 512 if W >= 2048 else 256
-            mx = {"heads": H, "dim": D, "rot_dim": 64, "vdim": D, "kv_rank": R, "scale": (D + 64) ** -0.5,
-                  "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
-            scfg = {"architecture": "Safolorn", "vocab": V, "width": W, "norm": {"eps": 1e-5},
-                    "layers": [{"type": "latent_attention", "mixer": mx, "mlp": {"kind": "dense", "ff": ff, "limit": 7.0}} for _ in range(nl)]}
-            seng = G.Engine(config=scfg, seed=7, dtype="bfloat16", max_tokens=ctx + n_dec + 64, page_size=64, max_portion=1024)
-            spf, spf_ops, sdec, sdc_ops, skernels, _ = _engine_times(G, seng, V, T, ctx, n_dec, BG_OPS)
-            s_params = nl * (W * (H * (D + 64) + R + 64) + W * H * D + 3.0 * ff * W)
-            s_flops, s_bytes = 2.0 * T * s_params + 2.0 * V * W, 2.0 * (s_params + V * W)
-            s_attn = 2.0 * nl * H * (2 * R + 64) * T * (T + 1) / 2
-            s_cache = 2.0 * nl * ctx * (R + 64)
-            rec["safolorn_equal_size"] = {
-                "config": {"kv_rank": R, "rot_dim": 64, "weight_bytes": seng.stats()["weight_bytes"]},
-                "prefill": {"tokens_per_s": T / spf, "ms": 1e3 * spf, "op_ms": spf_ops, "linear_tflops": s_flops / (spf_ops["op_linear"] / 1e3) / 1e12,
-                            "linear_frac_of_tensor_peak": s_flops / (spf_ops["op_linear"] / 1e3) / 1e12 / peaks["bf16_tflops_sustained"],
-                            "attn_tflops_cuda_cores": s_attn / (spf_ops["op_attn"] / 1e3) / 1e12},
-                "decode": {"tokens_per_s": 1.0 / sdec, "us_per_token": 1e6 * sdec, "kernels_per_token": skernels, "op_us": {k: 1e3 * v for k, v in sdc_ops.items()},
-                           "linear_gbs": s_bytes / (sdc_ops["op_linear"] / 1e3) / 1e9, "linear_frac_of_hbm_peak": s_bytes / (sdc_ops["op_linear"] / 1e3) / 1e9 / peaks["hbm_gbs"],
-                           "attn_gbs": s_cache / (sdc_ops["op_attn"] / 1e3) / 1e9,
-                           "token_frac_of_hbm_roofline": ((s_bytes + s_cache) / (peaks["hbm_gbs"] * 1e9)) / sdec},
-            }
-            seng.close()
+        if not args.no_sub_records:
+            rec["safolorn_equal_size"] = _safolorn_record(G, peaks, W, nl, H, D, ff, V, T, ctx, n_dec)
         records[size] = rec
     first = records[args.sizes.split(",")[0]]
     print(json.dumps({"metric": "begupel decode tokens/s", "value": first["decode"]["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
@@ -1103,12 +1109,109 @@ def run_kibilix(args):
                       "peaks": peaks, "sizes": records}), flush=True)
 
 
+TEZESUN_SIZES = {  # width, layers, heads, kv heads, size of one map, value size, window, kept tokens, latent heads, q_rank, kv_rank, rglru blocks, ff, vocab
+    "s": (1024, 9, 8, 2, 64, 128, 1024, 4, 8, 384, 256, 4, 4096, 32000),
+    "m": (2048, 9, 16, 4, 64, 128, 1024, 4, 16, 768, 512, 8, 8192, 32000),
+    "l": (4096, 6, 32, 8, 64, 128, 2048, 4, 32, 1536, 512, 16, 12288, 32000),
+}
+TZ_OPS = ("op_linear", "op_attn", "op_attn_latent", "op_attn_prep", "op_attn_expand", "op_attn_out", "op_conv", "op_gates", "op_recurrence", "op_residual", "op_rows")
+
+
+def tezesun_config(size):
+    """Layers in turn: a gated linear recurrence as wide as the model, differential attention over a window, latent attention
+    over everything; a dense feed-forward in each."""
+    W, L, H, Gk, D, Dv, win, keep, Hl, Rq, R, nb, ff, V = TEZESUN_SIZES[size]
+    kinds = [("rglru", {"width": W, "blocks": nb, "conv": 4}),
+             ("attention", {"heads": H, "kv_heads": Gk, "dim": D, "vdim": Dv, "scale": D ** -0.5, "softcap": 30.0, "diff": 0.6, "mask": {"size": win, "keep_first": keep},
+                            "rot": {"base": 500000.0, "dims": D, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}),
+             ("latent_attention", {"heads": Hl, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": R, "q_rank": Rq, "scale": 192 ** -0.5, "rot": {"base": 1000000.0, "dims": 64}})]
+    return {"architecture": "Tezesun", "vocab": V, "width": W, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+            "layers": [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": {"kind": "dense", "ff": ff}} for i in range(L)]}
+
+
+def run_tezesun(args):
+    """--arch tezesun: prefill and decode throughput of the Tezesun design (random bf16 weights) at layer sizes of real
+    models, through the serving engine (host call: H2D token ids, operator launches / graph replay, D2H result), with
+    cudaEvent time per operator class and roofline fractions; beside it Begupel (the same engine, products, window attention
+    kernels and a recurrence) and Safolorn (the latent attention kernels) at the same width, depth, heads and feed-forward."""
+    import gemma_ggml_b200 as G
+    G.init(0)
+    peaks = {"hbm_gbs": 6650.0, "bf16_tflops_sustained": 1400.0, "source": "fallback"}
+    try:
+        pk = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
+        peaks = {"hbm_gbs": float(pk["hbm_gbs"]), "bf16_tflops_sustained": float(pk["bf16_tflops_sustained"]), "source": "MEASURED_PEAKS.json"}
+    except Exception:
+        pass
+    T, ctx, n_dec = args.prefill_tokens if args.prefill_tokens != 512 else 2048, args.ctx, min(args.steps, 128)
+    records = {}
+    for size in args.sizes.split(","):
+        cfg = tezesun_config(size)
+        W, nl, H, Gk, D, Dv, win, keep, Hl, Rq, R, nb, ff, V = TEZESUN_SIZES[size]
+        eng = G.Engine(config=cfg, seed=7, dtype="bfloat16", max_tokens=ctx + n_dec + 64, page_size=64, max_portion=1024)
+        pf, pf_ops, dec, dc_ops, kernels, clocks = _engine_times(G, eng, V, T, ctx, n_dec, TZ_OPS)
+        wbytes = eng.stats()["weight_bytes"]
+        eng.close()
+        lin_params = uk_params = attn_flops = latent_flops = gate_flops = 0.0
+        cache_bytes = latent_bytes = rec_bytes = rec_step_bytes = 0.0
+        visible = float(sum(min(i + 1, win + keep) for i in range(T)))
+        for Ly in cfg["layers"]:
+            if Ly["type"] == "attention":
+                lin_params += W * (2 * H * D + 2 * Gk * D + Gk * Dv + H * Dv) + W * H * Dv
+                attn_flops += 4.0 * H * (D + Dv) * visible          # two maps: scores and weighted sum
+                cache_bytes += 2.0 * min(ctx, win + keep) * Gk * (2 * D + Dv)
+            elif Ly["type"] == "latent_attention":
+                lin_params += W * (Rq + R + 64) + Hl * 192 * Rq + W * Hl * 128
+                uk_params += Hl * 256.0 * R                          # absorbed in steps, expanded once per portion
+                latent_flops += 2.0 * Hl * (192 + 128) * T * (T + 1) / 2
+                latent_bytes += 2.0 * ctx * (R + 64)
+            else:
+                lin_params += 3.0 * W * W
+                gate_flops += 2.0 * T * W * 2 * (W // nb)
+                rec_bytes += T * W * (2 * 4 + 4 + 4 + 2.0)           # scan: both gates, u, y in; the output in 16 bits
+                rec_step_bytes += 2.0 * 2 * W * (W // nb) + 4.0 * 12 * W
+            lin_params += 2.0 * ff * W
+        lin_flops = 2.0 * T * lin_params + 2.0 * V * W
+        lin_bytes = 2.0 * (lin_params + V * W)
+        res_bytes = nl * T * W * (4.0 * 4 + 4)                       # x and two outputs in, x out, h and its shifted form in 16 bits
+        n_exp = sum(range(1024, T + 1, 1024)) if T % 1024 == 0 else T
+        rec = {
+            "config": {"width": W, "layers": nl, "heads": H, "kv_heads": Gk, "dim": D, "vdim": Dv, "window": win, "keep_first": keep, "latent_heads": Hl,
+                       "q_rank": Rq, "kv_rank": R, "rglru_blocks": nb, "ff": ff, "vocab": V, "weight_bytes": wbytes},
+            "prefill": {"tokens": T, "tokens_per_s": T / pf, "ms": 1e3 * pf, "op_ms": pf_ops, "clocks": clocks,
+                        "linear_tflops": lin_flops / (pf_ops["op_linear"] / 1e3) / 1e12,
+                        "linear_frac_of_tensor_peak": lin_flops / (pf_ops["op_linear"] / 1e3) / 1e12 / peaks["bf16_tflops_sustained"],
+                        "diff_attn_tflops_cuda_cores": attn_flops / (pf_ops["op_attn"] / 1e3) / 1e12,
+                        "latent_attn_tflops_cuda_cores": latent_flops / (pf_ops["op_attn_latent"] / 1e3) / 1e12,
+                        "expand_tflops": 2.0 * n_exp * uk_params / (pf_ops["op_attn_expand"] / 1e3) / 1e12,
+                        "gates_tflops": 3.0 * gate_flops / (pf_ops["op_gates"] / 1e3) / 1e12,
+                        "scan_gbs": rec_bytes / (pf_ops["op_recurrence"] / 1e3) / 1e9,
+                        "residual_gbs": res_bytes / (pf_ops["op_residual"] / 1e3) / 1e9},
+            "decode": {"n_kv": ctx, "tokens_per_s": 1.0 / dec, "us_per_token": 1e6 * dec, "kernels_per_token": kernels, "op_us": {k: 1e3 * v for k, v in dc_ops.items()},
+                       "linear_gbs": lin_bytes / (dc_ops["op_linear"] / 1e3) / 1e9, "linear_frac_of_hbm_peak": lin_bytes / (dc_ops["op_linear"] / 1e3) / 1e9 / peaks["hbm_gbs"],
+                       "diff_attn_gbs": cache_bytes / (dc_ops["op_attn"] / 1e3) / 1e9, "latent_attn_gbs": latent_bytes / (dc_ops["op_attn_latent"] / 1e3) / 1e9,
+                       "recurrence_gbs": rec_step_bytes / (dc_ops["op_recurrence"] / 1e3) / 1e9,
+                       "token_frac_of_hbm_roofline": ((lin_bytes + 2.0 * uk_params + cache_bytes + latent_bytes + rec_step_bytes) / (peaks["hbm_gbs"] * 1e9)) / dec},
+        }
+        if not args.no_sub_records:
+            rec["begupel_equal_size"] = _begupel_record(G, peaks, (W, nl, H, Gk, Dv, win, H, max(Gk, H // 2), H, ff, V), T, ctx, n_dec)
+            rec["safolorn_equal_size"] = _safolorn_record(G, peaks, W, nl, Hl, 128, ff, V, T, ctx, n_dec)
+        records[size] = rec
+    first = records[args.sizes.split(",")[0]]
+    print(json.dumps({"metric": "tezesun decode tokens/s", "value": first["decode"]["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+                      "steps": n_dec, "warmup": 8, "ms_per_step": first["decode"]["us_per_token"] / 1e3, "higher_is_better": True,
+                      "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic (random bf16 weights of the configured sizes)",
+                      "config": {"workload": "Tezesun sizes " + args.sizes + ": prefill of %d tokens, greedy decode at n_kv %d, through the serving engine" % (T, ctx),
+                                 "l2": "weights of every size exceed the 126 MB L2"},
+                      "peaks": peaks, "sizes": records}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--arch", default="gemma", choices=["gemma", "safolorn", "begupel", "ditalorn", "kibilix"],
+    ap.add_argument("--arch", default="gemma", choices=["gemma", "safolorn", "begupel", "ditalorn", "kibilix", "tezesun"],
                     help="gemma: the headline workload (default); safolorn: throughput of the Safolorn design beside Gemma at equal size; "
-                         "begupel: throughput of the Begupel design beside Safolorn at equal size; ditalorn: the Ditalorn design beside Safolorn at equal size; kibilix: the Kibilix design beside Begupel at equal size")
-    ap.add_argument("--sizes", default="s,m,l", help="--arch safolorn / begupel / ditalorn / kibilix: which of the sizes s, m, l to run")
+                         "begupel: throughput of the Begupel design beside Safolorn at equal size; ditalorn: the Ditalorn design beside Safolorn at equal size; kibilix: the Kibilix design beside Begupel at equal size; "
+                         "tezesun: the Tezesun design beside Begupel and Safolorn at equal size")
+    ap.add_argument("--sizes", default="s,m,l", help="--arch safolorn / begupel / ditalorn / kibilix / tezesun: which of the sizes s, m, l to run")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=256)
     ap.add_argument("--warmup", type=int, default=16)
@@ -1134,6 +1237,8 @@ def main():
         run_ditalorn(args)
     elif args.arch == "kibilix":
         run_kibilix(args)
+    elif args.arch == "tezesun":
+        run_tezesun(args)
     elif args.mode == "prefill":
         run_prefill(args)
     else:

@@ -1046,10 +1046,37 @@ __device__ __forceinline__ float xielu_f32(float z, const xielu_args &x) {
     return z > 0.f ? fmaf(x.ap * z, z, 0.5f * z) : fmaf(x.an, expm1f(z) - z, 0.5f * z);
 }
 
-template <typename E>
-__global__ void xielu_rows_kernel(const float *__restrict__ x, int64_t n, xielu_args xa, E *__restrict__ y) {
-    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) y[i] = from_f32<E>(xielu_f32(x[i], xa));
+// V numbers (V = 4: a 16-byte store in fp32, 8 bytes in bf16) rounded into the matrices' type
+template <int V, typename E> __device__ __forceinline__ void store_vec(E *dst, const float (&v)[V]) {
+    if (V == 4 && sizeof(E) == 2) {
+        union {
+            uint2 u;
+            __nv_bfloat16 h[4];
+        } p;
+#pragma unroll
+        for (int c = 0; c < V; c++) p.h[c] = __float2bfloat16_rn(v[c]);
+        *reinterpret_cast<uint2 *>(dst) = p.u;
+    } else if (V == 4) {
+        *reinterpret_cast<float4 *>(dst) = make_float4(v[0], v[1 % V], v[2 % V], v[3 % V]);
+    } else {
+        dst[0] = from_f32<E>(v[0]);
+    }
+}
+
+template <typename E, int V>
+__global__ void __launch_bounds__(256) xielu_rows_kernel(const float *__restrict__ x, int64_t n, xielu_args xa, E *__restrict__ y) {
+    const int64_t i = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
+    if (i >= n) return; // n is a multiple of V
+    float v[V];
+    if (V == 4) {
+        const float4 v4 = *reinterpret_cast<const float4 *>(x + i);
+        v[0] = v4.x, v[1 % V] = v4.y, v[2 % V] = v4.z, v[3 % V] = v4.w;
+    } else {
+        v[0] = x[i];
+    }
+#pragma unroll
+    for (int c = 0; c < V; c++) v[c] = xielu_f32(v[c], xa);
+    store_vec<V>(y + i, v);
 }
 
 // one of two mat-vecs that share a launch
@@ -1172,9 +1199,12 @@ __global__ void __launch_bounds__(TB) shift_norm_kernel(shift_norm_args<E> p, in
     if (p.rows) {
         const int64_t o = blockIdx.x;
         const float r = row(p.rows[o], o, false);
-        for (int64_t i = (int64_t)threadIdx.x * V; i < W; i += (int64_t)TB * V)
+        for (int64_t i = (int64_t)threadIdx.x * V; i < W; i += (int64_t)TB * V) {
+            float h[V];
 #pragma unroll
-            for (int c = 0; c < V; c++) p.h[o * W + i + c] = from_f32<E>(cur[i + c] * r * p.nw[i + c]);
+            for (int c = 0; c < V; c++) h[c] = cur[i + c] * r * p.nw[i + c];
+            store_vec<V>(p.h + o * W + i, h);
+        }
         return;
     }
     const int64_t t0 = (int64_t)blockIdx.x * nt, t1 = min(p.T, t0 + nt);
@@ -1188,14 +1218,17 @@ __global__ void __launch_bounds__(TB) shift_norm_kernel(shift_norm_args<E> p, in
         const float r = row(t, t, p.x_out != nullptr);
         if (!p.nw) continue;
         for (int64_t i = (int64_t)threadIdx.x * V; i < W; i += (int64_t)TB * V) {
+            float h[V], hs[V];
 #pragma unroll
-            for (int c = 0; c < V; c++) {
-                const float h = cur[i + c] * r * p.nw[i + c];
-                if (p.h) p.h[t * W + i + c] = from_f32<E>(h);
-                if (p.mu) {
-                    p.hs[t * W + i + c] = from_f32<E>(fmaf(before[i + c] - h, p.mu[i + c], h));
-                    before[i + c] = h;
+            for (int c = 0; c < V; c++) h[c] = cur[i + c] * r * p.nw[i + c];
+            if (p.h) store_vec<V>(p.h + t * W + i, h);
+            if (p.mu) {
+#pragma unroll
+                for (int c = 0; c < V; c++) {
+                    hs[c] = fmaf(before[i + c] - h[c], p.mu[i + c], h[c]);
+                    before[i + c] = h[c];
                 }
+                store_vec<V>(p.hs + t * W + i, hs);
             }
         }
     }
@@ -1215,7 +1248,8 @@ __global__ void __launch_bounds__(TB) shift_norm_kernel(shift_norm_args<E> p, in
 template <typename E>
 int shift_norm_launch(const shift_norm_args<E> &p) {
     const size_t smem = (size_t)p.W * 8;
-    const bool vec = p.W % 4 == 0 && (((uintptr_t)p.x | (uintptr_t)p.a | (uintptr_t)p.ls_a | (uintptr_t)p.b | (uintptr_t)p.ls_b | (uintptr_t)p.x_out) & 15) == 0;
+    const bool vec = p.W % 4 == 0 && (((uintptr_t)p.x | (uintptr_t)p.a | (uintptr_t)p.ls_a | (uintptr_t)p.b | (uintptr_t)p.ls_b | (uintptr_t)p.x_out |
+                                       (uintptr_t)p.h | (uintptr_t)p.hs) & 15) == 0;
     // tokens per CTA: the row before is computed again once per CTA, so as many as leave two CTAs for every SM
     int nt = 1;
     while (!p.rows && nt < 8 && p.T >= (int64_t)nt * 4 * ggb_sm_count()) nt *= 2;
@@ -1245,9 +1279,15 @@ int ggb_op_xielu_rows(int dt, const float *x, int64_t n, float ap, float an, voi
     GGB_REQUIRE_INIT();
     GGB_CHECK_DT(dt);
     GGB_CHECK_ARG(x && y && n > 0, "xielu_rows: bad arguments");
-    const unsigned blocks = (unsigned)((n + 255) / 256);
-    if (dt == GGB_TYPE_BF16) xielu_rows_kernel<<<blocks, 256, 0, ggb_cuda_stream()>>>(x, n, xielu_args{ap, an}, (__nv_bfloat16 *)y);
-    else xielu_rows_kernel<<<blocks, 256, 0, ggb_cuda_stream()>>>(x, n, xielu_args{ap, an}, (float *)y);
+    const bool vec = n % 4 == 0 && (((uintptr_t)x | (uintptr_t)y) & 15) == 0;
+    const unsigned blocks = (unsigned)((n / (vec ? 4 : 1) + 255) / 256);
+#define XR_LAUNCH(E, V) xielu_rows_kernel<E, V><<<blocks, 256, 0, ggb_cuda_stream()>>>(x, n, xielu_args{ap, an}, (E *)y);
+    if (dt == GGB_TYPE_BF16) {
+        if (vec) XR_LAUNCH(__nv_bfloat16, 4) else XR_LAUNCH(__nv_bfloat16, 1)
+    } else {
+        if (vec) XR_LAUNCH(float, 4) else XR_LAUNCH(float, 1)
+    }
+#undef XR_LAUNCH
     GGB_LAUNCH_CHECK();
     return GGB_OK;
 }

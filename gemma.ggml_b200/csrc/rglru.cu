@@ -176,17 +176,26 @@ __global__ void __launch_bounds__(128) rglru_conv_kernel(rglru_conv_args cv, int
         for (int j = 0; j < kMaxTaps - 1; j++) win[j] = j < nt ? cv.x[(t0 - nt + j) * cv.ld + c] + xb : 0.f; // kConvTokens > taps
     }
     const int64_t b = c / d, k = c - b * d;
-    for (int64_t t = t0; t < t1; t++) {
-        const float v = conv_tap(wt, win, nt, cv.x[t * cv.ld + c] + xb, wb);
-        u[t * C + c] = v;
-        if (split) {
-            __nv_bfloat16 *row = split + (b * T + t) * 3 * d + k;
-            const __nv_bfloat16 hi = __float2bfloat16_rn(v);
-            const float r1 = v - __bfloat162float(hi);
-            const __nv_bfloat16 mid = __float2bfloat16_rn(r1);
-            row[0] = hi;
-            row[d] = mid;
-            row[2 * d] = __float2bfloat16_rn(r1 - __bfloat162float(mid));
+    constexpr int kAhead = 8; // inputs of eight tokens in flight together
+    for (int64_t tb = t0; tb < t1; tb += kAhead) {
+        float xv[kAhead];
+#pragma unroll
+        for (int s = 0; s < kAhead; s++) xv[s] = cv.x[min(tb + s, t1 - 1) * cv.ld + c] + xb;
+#pragma unroll
+        for (int s = 0; s < kAhead; s++) {
+            const int64_t t = tb + s;
+            if (t >= t1) break;
+            const float v = conv_tap(wt, win, nt, xv[s], wb);
+            u[t * C + c] = v;
+            if (split) {
+                __nv_bfloat16 *row = split + (b * T + t) * 3 * d + k;
+                const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+                const float r1 = v - __bfloat162float(hi);
+                const __nv_bfloat16 mid = __float2bfloat16_rn(r1);
+                row[0] = hi;
+                row[d] = mid;
+                row[2 * d] = __float2bfloat16_rn(r1 - __bfloat162float(mid));
+            }
         }
     }
     if (t0 == 0)
@@ -392,7 +401,7 @@ int ggb_op_rglru_scan(int dt, const float *z, const float *u, const float *y, in
 #define SC_CH(E)                                               \
     {                                                          \
         if (C >= 32 * (int64_t)ggb_sm_count()) { SC_LAUNCH(E, 32) } \
-        else if (C >= 16 * (int64_t)ggb_sm_count()) { SC_LAUNCH(E, 16) } \
+        else if (C >= 12 * (int64_t)ggb_sm_count()) { SC_LAUNCH(E, 16) } \
         else { SC_LAUNCH(E, 8) }                               \
     }
     if (dt == GGB_TYPE_BF16) SC_CH(__nv_bfloat16) else SC_CH(float)

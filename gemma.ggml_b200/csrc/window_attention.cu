@@ -390,14 +390,14 @@ __global__ void __launch_bounds__(32) window_merge_kernel(const float *__restric
     for (int a = 0; a < MAPS; a++) {
         const float *pp = part + (t * H + h) * n_split * pw + a * kPartW;
         float M = -INFINITY;
+#pragma unroll 4
         for (int s = 0; s < n_split; s++) M = fmaxf(M, pp[s * pw]);
         l[a] = 0.f;
 #pragma unroll
         for (int r = 0; r < kMaxDvRegs; r++) acc[a][r] = 0.f;
-        for (int s = 0; s < n_split; s++) {
-            const float ms = pp[s * pw];
-            if (ms == -INFINITY) continue;
-            const float f = expf(ms - M);
+#pragma unroll 4
+        for (int s = 0; s < n_split; s++) { // a split without keys holds m = -inf and zeros: its weight is 0; the loads do not wait for it
+            const float f = expf(pp[s * pw] - M);
             l[a] = fmaf(pp[s * pw + 1], f, l[a]);
 #pragma unroll
             for (int r = 0; r < kMaxDvRegs; r++) acc[a][r] = fmaf(pp[s * pw + 2 + r * 32 + lane], f, acc[a][r]);
