@@ -198,6 +198,12 @@ _CUDA_SIG = {
     "ggb_op_latent_expand_rot": (i32, [i32, vp, vp, i32, i64, i64, i32, i32, i32, i32, i32, vp, vp, vp, vp, i64]),
     "ggb_op_latent_q_rotate": (i32, [vp, i64, i64, i32, i32, i32, i32, i32, vp, vp, f32, vp]),
     "ggb_op_hyper_mix_moe": (i32, [i32, vp, vp, vp, vp, vp, i64, i32, i32, i32, vp, vp, vp, i32, vp, vp, f32, i64, i64, vp, vp, vp]),
+    "ggb_op_linear_act": (i32, [i32, vp, i64, i64, vp, i64, i64, i32, vp]),
+    "ggb_op_residual_layer_norm": (i32, [i32, vp, vp, vp, vp, vp, i64, i32, i32, vp, vp, i64, vp, vp, vp, vp, vp, f32, i64, i64, vp, vp, vp]),
+    "ggb_op_head_qkv_store": (i32, [i32, vp, vp, vp, i64, i64, i32, i32, i32, i32, vp, vp, f32, i32, i32, vp, f32, vp, vp, i32, vp, vp]),
+    "ggb_op_masked_attn_gated": (i32, [i32, vp, vp, vp, i32, vp, i64, i32, i32, i32, i32, i64, i64, f32, vp, vp, i64, vp, vp]),
+    "ggb_op_moe_route_softmax_groups": (i32, [i32, vp, i64, i64, vp, vp, i32, i32, i32, i32, i32, f32, vp, vp, vp, vp]),
+    "ggb_op_moe_linear_shared": (i32, [i32, vp, i64, i64, vp, i64, i32, i64, i32, i32, vp, i32, vp, i64, vp, i64, i64, vp, i64, vp]),
     "ggb_comm_unique_id": (i32, [vp]), "ggb_comm_init": (i32, [vp, i32, i32]), "ggb_comm_destroy": (i32, []),
     "ggb_comm_rank": (i32, []), "ggb_comm_size": (i32, []), "ggb_op_allgather": (i32, [vp, vp, sz]),
 }
@@ -240,6 +246,7 @@ _HOST_SIG = {
     "dl_config_probe": (i32, [C.c_char_p, P(i64)]),
     "kb_config_probe": (i32, [C.c_char_p, P(i64)]),
     "tz_config_probe": (i32, [C.c_char_p, P(i64)]),
+    "fk_config_probe": (i32, [C.c_char_p, P(i64)]),
     "st_probe": (i32, [C.c_char_p, C.c_char_p, P(i64), P(i64), C.c_char_p, i32, P(i64)]),
     "mul_mat": (None, [i64, i64, i64, i64, i64, i64, i64, sz, i64, vp, vp, vp, vp, i32, vp]),
     "init_cuda_offload": (i32, [i32]),

@@ -50,7 +50,7 @@ __device__ __forceinline__ void vec_row_dot(const E *__restrict__ wr, const E *_
     }
 }
 
-// ACT 1: the output is relu(.)^2 in the matrices' type (c_act) instead of fp32 (c)
+// ACT: the output is act(.) in the matrices' type (c_act) instead of fp32 (c)
 template <typename E, int TT, int ACT = 0>
 __global__ void __launch_bounds__(256) linear_vec_kernel(const E *__restrict__ w, int64_t N, int64_t K, const E *__restrict__ a,
                                                          int64_t lda, float *__restrict__ c, int64_t ldc, E *__restrict__ c_act = nullptr) {
@@ -66,7 +66,7 @@ __global__ void __launch_bounds__(256) linear_vec_kernel(const E *__restrict__ w
     for (int t = 0; t < TT; t++) {
         const float s = warp_sum_f32(acc[t]);
         if (lane == 0) {
-            if (ACT == 1) c_act[t * ldc + n] = from_f32<E>(s > 0.f ? s * s : 0.f);
+            if (ACT) c_act[t * ldc + n] = from_f32<E>(act_f32(s, ACT));
             else c[t * ldc + n] = s;
         }
     }
@@ -133,9 +133,8 @@ __global__ void __launch_bounds__(256) linear_tile_kernel(const E *__restrict__ 
             const int64_t n = n0 + tx * 4 + j;
             if (n >= N) continue;
             float v = acc[i][j];
-            if (ACT == 1) { // square of relu, stored in the matrices' type (the next product's operand)
-                v = v > 0.f ? v * v : 0.f;
-                c_act[m * ldc + n] = from_f32<E>(v);
+            if (ACT) { // stored in the matrices' type (the next product's operand)
+                c_act[m * ldc + n] = from_f32<E>(act_f32(v, ACT));
             } else {
                 c[m * ldc + n] = v;
             }
@@ -342,20 +341,20 @@ int linear_launch(const E *w, int64_t N, int64_t K, const E *a, int64_t lda, int
     return GGB_OK;
 }
 
-// y (E, [T][N]) = relu(a W^T)^2 in one launch: the mat-vec or the tile kernel with the activation as its epilogue
-template <typename E>
-int linear_relu2_launch(const E *w, int64_t N, int64_t K, const E *a, int64_t lda, int64_t T, E *y) {
+// y (E, [T][N]) = act(a W^T) in one launch: the mat-vec or the tile kernel with the activation as its epilogue
+template <typename E, int ACT>
+int linear_act_launch(const E *w, int64_t N, int64_t K, const E *a, int64_t lda, int64_t T, E *y) {
     cudaStream_t st = ggb_cuda_stream();
     if (T <= kVecT) {
         const dim3 grid((unsigned)((N + 7) / 8));
         switch ((int)T) {
-#define VEC_CASE(TT) case TT: linear_vec_kernel<E, TT, 1><<<grid, 256, 0, st>>>(w, N, K, a, lda, nullptr, N, y); break;
+#define VEC_CASE(TT) case TT: linear_vec_kernel<E, TT, ACT><<<grid, 256, 0, st>>>(w, N, K, a, lda, nullptr, N, y); break;
             VEC_CASE(1) VEC_CASE(2) VEC_CASE(3) VEC_CASE(4) VEC_CASE(5) VEC_CASE(6) VEC_CASE(7) VEC_CASE(8)
 #undef VEC_CASE
         }
     } else {
         const dim3 grid((unsigned)((N + 63) / 64), (unsigned)((T + 63) / 64));
-        linear_tile_kernel<E, false, 1><<<grid, 256, 0, st>>>(w, N, K, a, lda, T, nullptr, y, N, ggb_moe_groups{});
+        linear_tile_kernel<E, false, ACT><<<grid, 256, 0, st>>>(w, N, K, a, lda, T, nullptr, y, N, ggb_moe_groups{});
     }
     GGB_LAUNCH_CHECK();
     return GGB_OK;
@@ -369,7 +368,8 @@ int ggb_linear_grouped_launch(int dt, const void *w, int64_t N, int64_t K, const
     cudaStream_t st = ggb_cuda_stream();
     const dim3 grid((unsigned)((N + 63) / 64), (unsigned)max_tiles);
 #define GRP_CASE(E)                                                                                                           \
-    if (act) linear_tile_kernel<E, true, 1><<<grid, 256, 0, st>>>((const E *)w, N, K, (const E *)a, lda, 0, nullptr, (E *)c_act, ldc, grp); \
+    if (act == GGB_ACT_GELU_ERF) linear_tile_kernel<E, true, GGB_ACT_GELU_ERF><<<grid, 256, 0, st>>>((const E *)w, N, K, (const E *)a, lda, 0, nullptr, (E *)c_act, ldc, grp); \
+    else if (act) linear_tile_kernel<E, true, GGB_ACT_RELU2><<<grid, 256, 0, st>>>((const E *)w, N, K, (const E *)a, lda, 0, nullptr, (E *)c_act, ldc, grp); \
     else linear_tile_kernel<E, true, 0><<<grid, 256, 0, st>>>((const E *)w, N, K, (const E *)a, lda, 0, c, nullptr, ldc, grp);
     if (dt == GGB_TYPE_BF16) { GRP_CASE(__nv_bfloat16) } else { GRP_CASE(float) }
 #undef GRP_CASE
@@ -670,16 +670,6 @@ int ggb_op_norm_gate(int dt, const float *o, int64_t ldo, const float *gate, int
 // ------------------------------------------------------------------------------------------------ learned positions, norms on both sides of a sublayer
 namespace {
 
-__device__ __forceinline__ float block_sum_any(float v, float *red) { // all threads get the sum; blockDim.x a multiple of 32, at most 1024
-    v = warp_sum_f32(v);
-    __syncthreads(); // `red` may still be read by the previous call
-    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-    __syncthreads();
-    float tot = 0.f;
-    for (int i = 0; i < (int)(blockDim.x >> 5); i++) tot += red[i];
-    return tot;
-}
-
 // one CTA per token: the embedding row times `scale` plus the (unscaled) row of the token's position
 template <typename E>
 __global__ void __launch_bounds__(256) embed_pos_kernel(const E *__restrict__ table, const E *__restrict__ pos_table, const int32_t *__restrict__ ids,
@@ -936,15 +926,13 @@ __global__ void __launch_bounds__(TB) hyper_mix_kernel(float *xs, const float *_
         for (int c = 0; c < V; c++) h[b * W + i + c] = from_f32<E>(hm_row[i + c] * r * nw[i + c]);
 }
 
-// y (dt, dense [T][F]) = act(x) for fp32 rows of stride ldx; act 0: as it is, 1: the square of relu
+// y (dt, dense [T][F]) = act(x) for fp32 rows of stride ldx (GGB_ACT_*)
 template <typename E>
 __global__ void act_rows_kernel(const float *__restrict__ x, int64_t ldx, int64_t T, int64_t F, int act, E *__restrict__ y) {
     const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= T * F) return;
     const int64_t t = i / F, f = i - t * F;
-    float v = x[t * ldx + f];
-    if (act == 1) v = v > 0.f ? v * v : 0.f;
-    y[i] = from_f32<E>(v);
+    y[i] = from_f32<E>(act_f32(x[t * ldx + f], act));
 }
 
 } // namespace
@@ -1018,14 +1006,30 @@ int ggb_op_linear_relu2(int dt, const void *w, int64_t N, int64_t K, const void 
         const int rc = ggb_gemm_dense_bf16(w, N, K, a, T, scratch, N);
         return rc ? rc : ggb_op_act_rows(dt, scratch, N, T, N, 1, y);
     }
-    if (dt == GGB_TYPE_BF16) return linear_relu2_launch((const __nv_bfloat16 *)w, N, K, (const __nv_bfloat16 *)a, lda, T, (__nv_bfloat16 *)y);
-    return linear_relu2_launch((const float *)w, N, K, (const float *)a, lda, T, (float *)y);
+    if (dt == GGB_TYPE_BF16)
+        return linear_act_launch<__nv_bfloat16, GGB_ACT_RELU2>((const __nv_bfloat16 *)w, N, K, (const __nv_bfloat16 *)a, lda, T, (__nv_bfloat16 *)y);
+    return linear_act_launch<float, GGB_ACT_RELU2>((const float *)w, N, K, (const float *)a, lda, T, (float *)y);
+}
+
+int ggb_op_linear_act(int dt, const void *w, int64_t N, int64_t K, const void *a, int64_t lda, int64_t T, int act, void *y) {
+    GGB_REQUIRE_INIT();
+    GGB_CHECK_DT(dt);
+    GGB_CHECK_ARG(w && a && y && N > 0 && K > 0 && T > 0 && lda >= K, "linear_act: bad shape N=%lld K=%lld T=%lld", (long long)N, (long long)K, (long long)T);
+    GGB_CHECK_ARG(act == GGB_ACT_RELU2 || act == GGB_ACT_GELU_ERF, "linear_act: activation %d", act);
+    if (dt == GGB_TYPE_BF16 && lda == K && N % 8 == 0 && ((uintptr_t)y & 15) == 0 && ggb_gemm_dense_bf16_fits(N, K, T, N))
+        return ggb_gemm_dense_bf16(w, N, K, a, T, nullptr, N, y, act);
+#define LA_CASE(E)                                                                                                                          \
+    return act == GGB_ACT_RELU2 ? linear_act_launch<E, GGB_ACT_RELU2>((const E *)w, N, K, (const E *)a, lda, T, (E *)y)                      \
+                                : linear_act_launch<E, GGB_ACT_GELU_ERF>((const E *)w, N, K, (const E *)a, lda, T, (E *)y);
+    if (dt == GGB_TYPE_BF16) LA_CASE(__nv_bfloat16)
+    LA_CASE(float)
+#undef LA_CASE
 }
 
 int ggb_op_act_rows(int dt, const float *x, int64_t ldx, int64_t T, int64_t F, int act, void *y) {
     GGB_REQUIRE_INIT();
     GGB_CHECK_DT(dt);
-    GGB_CHECK_ARG(x && y && T > 0 && F > 0 && ldx >= F && (act == 0 || act == 1), "act_rows: bad arguments");
+    GGB_CHECK_ARG(x && y && T > 0 && F > 0 && ldx >= F && (act == GGB_ACT_NONE || act == GGB_ACT_RELU2 || act == GGB_ACT_GELU_ERF), "act_rows: bad arguments");
     const unsigned blocks = (unsigned)((T * F + 255) / 256);
     if (dt == GGB_TYPE_BF16) act_rows_kernel<<<blocks, 256, 0, ggb_cuda_stream()>>>(x, ldx, T, F, act, (__nv_bfloat16 *)y);
     else act_rows_kernel<<<blocks, 256, 0, ggb_cuda_stream()>>>(x, ldx, T, F, act, (float *)y);
@@ -1044,23 +1048,6 @@ struct xielu_args {
 // z > 0: ap z^2 + z / 2; z <= 0: an (exp(z) - 1 - z) + z / 2
 __device__ __forceinline__ float xielu_f32(float z, const xielu_args &x) {
     return z > 0.f ? fmaf(x.ap * z, z, 0.5f * z) : fmaf(x.an, expm1f(z) - z, 0.5f * z);
-}
-
-// V numbers (V = 4: a 16-byte store in fp32, 8 bytes in bf16) rounded into the matrices' type
-template <int V, typename E> __device__ __forceinline__ void store_vec(E *dst, const float (&v)[V]) {
-    if (V == 4 && sizeof(E) == 2) {
-        union {
-            uint2 u;
-            __nv_bfloat16 h[4];
-        } p;
-#pragma unroll
-        for (int c = 0; c < V; c++) p.h[c] = __float2bfloat16_rn(v[c]);
-        *reinterpret_cast<uint2 *>(dst) = p.u;
-    } else if (V == 4) {
-        *reinterpret_cast<float4 *>(dst) = make_float4(v[0], v[1 % V], v[2 % V], v[3 % V]);
-    } else {
-        dst[0] = from_f32<E>(v[0]);
-    }
 }
 
 template <typename E, int V>

@@ -83,6 +83,17 @@ __global__ void __launch_bounds__(32) moe_select_kernel(const float *__restrict_
     }
 }
 
+// one warp: the choice scores of every group but the `keep` best ones (larger score, then lower index) become -inf
+__device__ __forceinline__ void drop_groups_warp(float *ch, const float *gsc, int gs, int n_groups, int keep, int lane) {
+    for (int g = lane; g < n_groups; g += 32) {
+        int before = 0;
+        for (int o = 0; o < n_groups; o++) before += (gsc[o] > gsc[g]) || (gsc[o] == gsc[g] && o < g);
+        if (before >= keep)
+            for (int e = g * gs; e < (g + 1) * gs; e++) ch[e] = -INFINITY;
+    }
+    __syncwarp();
+}
+
 // one warp per token, sigmoid scores with a choice correction and groups: s = sigmoid(z); the choice score of expert e is
 // s_e + corr_e; the experts form n_groups equal groups of neighbours, a group's score is the sum of its two largest
 // choice scores, and only experts of the `keep` best groups (ties: the lower group) can be chosen; among them the `top`
@@ -108,14 +119,7 @@ __device__ __forceinline__ void select_sigmoid_warp(float *sc, float *ch, float 
             gsc[g] = gs > 1 ? a + b : a;
         }
         __syncwarp();
-        // a group stays when fewer than `keep` groups come before it in the order (larger score, then lower index)
-        for (int g = lane; g < n_groups; g += 32) {
-            int before = 0;
-            for (int o = 0; o < n_groups; o++) before += (gsc[o] > gsc[g]) || (gsc[o] == gsc[g] && o < g);
-            if (before >= keep)
-                for (int e = g * gs; e < (g + 1) * gs; e++) ch[e] = -INFINITY;
-        }
-        __syncwarp();
+        drop_groups_warp(ch, gsc, gs, n_groups, keep, lane);
     }
     for (int k = 0; k < top; k++) {
         float bv = -INFINITY;
@@ -131,6 +135,7 @@ __device__ __forceinline__ void select_sigmoid_warp(float *sc, float *ch, float 
             if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
         }
         if (lane == 0) {
+            if (bi >= n_exp) bi = 0; // logits that are no numbers: any expert, but one that exists
             idx[t * top + k] = bi;
             wt[t * top + k] = sc[bi];
             sc[bi] = -1.0f; // taken: a score is never negative otherwise
@@ -139,11 +144,13 @@ __device__ __forceinline__ void select_sigmoid_warp(float *sc, float *ch, float 
     }
 }
 
-// one warp per token, soft-max scores over ALL experts with a choice correction: s = softmax(z); the `top` largest
-// s_e + corr_e win (ties: the lower index); the weight of a chosen expert is its s divided by the chosen ones' sum
-// (+ 1e-20).  sc holds the logits on entry (the scores afterwards), ch is scratch.
-__device__ __forceinline__ void select_softmax_warp(float *sc, float *ch, const float *__restrict__ corr, int n_exp, int top, int64_t t, int lane,
-                                                    int32_t *__restrict__ idx, float *__restrict__ wt) {
+// one warp per token, soft-max scores over ALL experts with a choice correction and groups: s = softmax(z); the choice score
+// of expert e is s_e + corr_e; the experts form n_groups equal groups of neighbours, a group's score is its largest choice
+// score and only experts of the `keep` best groups (ties: the lower group) can be chosen; the `top` largest win (ties: the
+// lower index); the weight of a chosen expert is its s divided by the chosen ones' sum (+ 1e-20), times scale.  sc holds the
+// logits on entry (the scores afterwards), ch and gsc are scratch.
+__device__ __forceinline__ void select_softmax_warp(float *sc, float *ch, float *gsc, const float *__restrict__ corr, int n_exp, int top, int n_groups,
+                                                    int keep, float scale, int64_t t, int lane, int32_t *__restrict__ idx, float *__restrict__ wt) {
     float m = -INFINITY;
     for (int e = lane; e < n_exp; e += 32) m = fmaxf(m, sc[e]);
     m = warp_max_f32(m);
@@ -160,6 +167,16 @@ __device__ __forceinline__ void select_softmax_warp(float *sc, float *ch, const 
         ch[e] = p + (corr ? corr[e] : 0.f);
     }
     __syncwarp();
+    if (keep < n_groups) {
+        const int gs = n_exp / n_groups;
+        for (int g = lane; g < n_groups; g += 32) {
+            float a = -INFINITY;
+            for (int e = g * gs; e < (g + 1) * gs; e++) a = fmaxf(a, ch[e]);
+            gsc[g] = a;
+        }
+        __syncwarp();
+        drop_groups_warp(ch, gsc, gs, n_groups, keep, lane);
+    }
     float chosen = 0.f; // lane 0: sum of the chosen scores, in slot order
     for (int k = 0; k < top; k++) {
         float bv = -INFINITY;
@@ -175,6 +192,7 @@ __device__ __forceinline__ void select_softmax_warp(float *sc, float *ch, const 
             if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
         }
         if (lane == 0) {
+            if (bi >= n_exp) bi = 0; // logits that are no numbers: any expert, but one that exists
             idx[t * top + k] = bi;
             wt[t * top + k] = sc[bi];
             chosen += sc[bi];
@@ -184,16 +202,16 @@ __device__ __forceinline__ void select_softmax_warp(float *sc, float *ch, const 
     }
     if (lane == 0) {
         chosen += 1e-20f;
-        for (int k = 0; k < top; k++) wt[t * top + k] = wt[t * top + k] / chosen;
+        for (int k = 0; k < top; k++) wt[t * top + k] = wt[t * top + k] / chosen * scale;
     }
 }
 
-__global__ void __launch_bounds__(32) moe_select_softmax_kernel(const float *__restrict__ zg, const float *__restrict__ corr, int n_exp, int top,
-                                                                int32_t *__restrict__ idx, float *__restrict__ wt) {
-    extern __shared__ float sm[]; // [n_exp] scores, [n_exp] choice scores
-    for (int e = threadIdx.x; e < n_exp; e += 32) sm[e] = zg[(int64_t)blockIdx.x * n_exp + e];
+__global__ void __launch_bounds__(32) moe_select_softmax_kernel(const float *__restrict__ zg, int64_t ldz, const float *__restrict__ corr, int n_exp, int top,
+                                                                int n_groups, int keep, float scale, int32_t *__restrict__ idx, float *__restrict__ wt) {
+    extern __shared__ float sm[]; // [n_exp] scores, [n_exp] choice scores, [n_groups] group scores
+    for (int e = threadIdx.x; e < n_exp; e += 32) sm[e] = zg[(int64_t)blockIdx.x * ldz + e];
     __syncwarp();
-    select_softmax_warp(sm, sm + n_exp, corr, n_exp, top, blockIdx.x, threadIdx.x, idx, wt);
+    select_softmax_warp(sm, sm + n_exp, sm + 2 * n_exp, corr, n_exp, top, n_groups, keep, scale, blockIdx.x, threadIdx.x, idx, wt);
 }
 
 __global__ void __launch_bounds__(32) moe_select_sigmoid_kernel(const float *__restrict__ zg, const float *__restrict__ corr, int n_exp, int top,
@@ -208,14 +226,15 @@ __global__ void __launch_bounds__(32) moe_select_sigmoid_kernel(const float *__r
 // each, so that the router's rows are read by many SMs; the CTA that finishes last for its token (a counter per token, put
 // back to zero by that CTA) reads all logits back and chooses.  With row_src the slots are also listed as the mat-vec form
 // of the grouped products reads them (slot s = row s: no order is needed there), which stands in for moe_group_kernel.
-// SOFTMAX: the rule of select_softmax_warp instead (n_groups and keep unused)
+// SOFTMAX: the rule of select_softmax_warp instead.  The matrix may have n_extra more rows behind the experts' (other numbers that
+// read the same input, a gate for instance): their products are left in the logits behind the experts' and choose nothing.
 constexpr int kRouteStepTokens = 32, kRouteStepWarps = 8;
 __device__ unsigned int g_route_done[kRouteStepTokens];
 
 template <typename E, bool SOFTMAX>
 __global__ void __launch_bounds__(32 * kRouteStepWarps) moe_route_sigmoid_step_kernel(const E *__restrict__ h, int64_t W, const float *__restrict__ w,
-                                                                     const float *__restrict__ corr, int n_exp, int top, int n_groups, int keep,
-                                                                     float *zg, int32_t *__restrict__ idx, float *__restrict__ wt,
+                                                                     const float *__restrict__ corr, int n_exp, int n_extra, int top, int n_groups, int keep,
+                                                                     float scale, float *zg, int32_t *__restrict__ idx, float *__restrict__ wt,
                                                                      int32_t *__restrict__ row_src, int32_t *__restrict__ inv,
                                                                      int32_t *__restrict__ row_expert) {
     extern __shared__ float sm[];
@@ -223,10 +242,11 @@ __global__ void __launch_bounds__(32 * kRouteStepWarps) moe_route_sigmoid_step_k
     const int64_t t = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int e = (int)blockIdx.y * kRouteStepWarps + warp;
-    if (e < n_exp) {
+    const int64_t ldz = n_exp + n_extra;
+    if (e < ldz) {
         const float s = router_dot(h + t * W, w + (int64_t)e * W, W, lane);
         if (lane == 0) {
-            zg[t * n_exp + e] = s;
+            zg[t * ldz + e] = s;
             __threadfence(); // the logit is visible before this CTA is counted
         }
     }
@@ -235,11 +255,11 @@ __global__ void __launch_bounds__(32 * kRouteStepWarps) moe_route_sigmoid_step_k
     __syncthreads();
     if (!last) return;
     __threadfence();
-    for (int i = threadIdx.x; i < n_exp; i += blockDim.x) sm[i] = __ldcg(zg + t * n_exp + i); // other CTAs wrote them: not through L1
+    for (int i = threadIdx.x; i < n_exp; i += blockDim.x) sm[i] = __ldcg(zg + t * ldz + i); // other CTAs wrote them: not through L1
     if (threadIdx.x == 0) g_route_done[t] = 0; // the next launch starts from zero
     __syncthreads();
     if (warp != 0) return;
-    if (SOFTMAX) select_softmax_warp(sm, sm + n_exp, corr, n_exp, top, t, lane, idx, wt);
+    if (SOFTMAX) select_softmax_warp(sm, sm + n_exp, sm + 2 * n_exp, corr, n_exp, top, n_groups, keep, scale, t, lane, idx, wt);
     else select_sigmoid_warp(sm, sm + n_exp, sm + 2 * n_exp, corr, n_exp, top, n_groups, keep, t, lane, idx, wt);
     __syncwarp();
     if (row_src)
@@ -298,6 +318,7 @@ __global__ void __launch_bounds__(256) moe_vec_kernel(const E *__restrict__ w, i
     const int row = blockIdx.y;
     if (n >= N || row_expert[row] >= n_real) return; // an expert without matrices: nothing to compute
     // ACT 2: an expert's matrix holds N gate rows, then N up rows; output n is silu(gate_n) * up_n
+    // (every other ACT: act_f32, one row per output)
     // ACT 3: the same rows; g = min(gate_n, limit), u = clamp(up_n, -limit, limit), output g * sigmoid(alpha g) * (u + 1)
     constexpr bool GATED = ACT == 2 || ACT == 3;
     const E *wr = w + ((int64_t)row_expert[row] * (GATED ? 2 * N : N) + n) * K;
@@ -327,7 +348,7 @@ __global__ void __launch_bounds__(256) moe_vec_kernel(const E *__restrict__ w, i
     acc = warp_sum_f32(acc);
     if (GATED) up = warp_sum_f32(up);
     if (lane == 0) {
-        if (ACT == 1) c_act[(int64_t)row * ldc + n] = from_f32<E>(acc > 0.f ? acc * acc : 0.f);
+        if (ACT == GGB_ACT_RELU2 || ACT == GGB_ACT_GELU_ERF) c_act[(int64_t)row * ldc + n] = from_f32<E>(act_f32(acc, ACT));
         else if (ACT == 2) c_act[(int64_t)row * ldc + n] = from_f32<E>(acc / (1.0f + expf(-acc)) * up);
         else if (ACT == 3) {
             const float g = fminf(acc, limit), u = fminf(fmaxf(up, -limit), limit);
@@ -335,6 +356,54 @@ __global__ void __launch_bounds__(256) moe_vec_kernel(const E *__restrict__ w, i
         }
         else c[(int64_t)row * ldc + n] = acc;
     }
+}
+
+// few slots, an expert that every token uses beside the chosen ones: rows n_slots .. n_slots + T - 1 of the grid are the tokens'
+// products with that expert's matrix, which has sizes of its own (one launch for both)
+template <typename E> struct shared_product {
+    const E *w, *a;
+    int64_t N, K, lda, ldc;
+    float *c;
+    E *c_act;
+    int vec;
+};
+template <typename E, int ACT>
+__global__ void __launch_bounds__(256) moe_vec_shared_kernel(const E *__restrict__ w, int64_t N, int64_t K, const E *__restrict__ a, int64_t lda,
+                                                             const int32_t *__restrict__ row_src, const int32_t *__restrict__ row_expert,
+                                                             float *__restrict__ c, E *__restrict__ c_act, int64_t ldc, int vec, int n_slots,
+                                                             shared_product<E> sh) {
+    constexpr int VE = 16 / (int)sizeof(E);
+    const int lane = threadIdx.x & 31;
+    const int64_t n = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+    const int row = blockIdx.y, t = row - n_slots;
+    const E *wr, *ar;
+    if (t < 0) {
+        if (n >= N) return;
+        wr = w + ((int64_t)row_expert[row] * N + n) * K;
+        ar = a + (int64_t)(row_src ? row_src[row] : row) * lda;
+    } else {
+        if (n >= sh.N) return;
+        wr = sh.w + n * sh.K;
+        ar = sh.a + t * sh.lda;
+        K = sh.K, vec = sh.vec;
+    }
+    float acc = 0.f;
+    if (vec) {
+#pragma unroll 4
+        for (int64_t k = (int64_t)lane * VE; k < K; k += 32 * VE) {
+            const uint4 wv = ldg_stream_u4(wr + k), av = *reinterpret_cast<const uint4 *>(ar + k);
+            const E *we = reinterpret_cast<const E *>(&wv), *ae = reinterpret_cast<const E *>(&av);
+#pragma unroll
+            for (int u = 0; u < VE; u++) acc = fmaf(to_f32(we[u]), to_f32(ae[u]), acc);
+        }
+    } else {
+        for (int64_t k = lane; k < K; k += 32) acc = fmaf(to_f32(wr[k]), to_f32(ar[k]), acc);
+    }
+    acc = warp_sum_f32(acc);
+    if (lane != 0) return;
+    const int64_t at = t < 0 ? row * ldc + n : t * sh.ldc + n;
+    if (ACT) (t < 0 ? c_act : sh.c_act)[at] = from_f32<E>(act_f32(acc, ACT));
+    else (t < 0 ? c : sh.c)[at] = acc;
 }
 
 // rows of A in sorted-slot order (the tensor-core product reads its operand contiguously): y[i] = a[row_src[i]], 16 bytes a thread
@@ -410,10 +479,10 @@ int ggb_op_moe_route_sigmoid(int dt, const void *h, int64_t W, int64_t T, const 
         const bool lists = ws && ggb_moe_step_form(n);
         int32_t *row_src = lists ? ws + n_exp + 1 : nullptr, *inv = lists ? row_src + n : nullptr, *row_expert = lists ? inv + n + 2 * mt + 1 : nullptr;
         if (dt == GGB_TYPE_BF16)
-            moe_route_sigmoid_step_kernel<__nv_bfloat16, false><<<dim3((unsigned)T, (unsigned)((n_exp + kRouteStepWarps - 1) / kRouteStepWarps)), 32 * kRouteStepWarps, smem, ggb_cuda_stream()>>>((const __nv_bfloat16 *)h, W, w_router, correction, n_exp, top, n_groups,
-                                                                                         keep, logits, idx, wt, row_src, inv, row_expert);
+            moe_route_sigmoid_step_kernel<__nv_bfloat16, false><<<dim3((unsigned)T, (unsigned)((n_exp + kRouteStepWarps - 1) / kRouteStepWarps)), 32 * kRouteStepWarps, smem, ggb_cuda_stream()>>>((const __nv_bfloat16 *)h, W, w_router, correction, n_exp, 0, top, n_groups,
+                                                                                         keep, 1.f, logits, idx, wt, row_src, inv, row_expert);
         else
-            moe_route_sigmoid_step_kernel<float, false><<<dim3((unsigned)T, (unsigned)((n_exp + kRouteStepWarps - 1) / kRouteStepWarps)), 32 * kRouteStepWarps, smem, ggb_cuda_stream()>>>((const float *)h, W, w_router, correction, n_exp, top, n_groups, keep,
+            moe_route_sigmoid_step_kernel<float, false><<<dim3((unsigned)T, (unsigned)((n_exp + kRouteStepWarps - 1) / kRouteStepWarps)), 32 * kRouteStepWarps, smem, ggb_cuda_stream()>>>((const float *)h, W, w_router, correction, n_exp, 0, top, n_groups, keep, 1.f,
                                                                                          logits, idx, wt, row_src, inv, row_expert);
         GGB_LAUNCH_CHECK();
         return GGB_OK;
@@ -432,32 +501,41 @@ int ggb_op_moe_route_sigmoid(int dt, const void *h, int64_t W, int64_t T, const 
 
 int ggb_op_moe_route_softmax(int dt, const void *h, int64_t W, int64_t T, const float *w_router, const float *correction, int n_exp, int top,
                              float *logits, int32_t *idx, float *wt, int32_t *ws) {
+    return ggb_op_moe_route_softmax_groups(dt, h, W, T, w_router, correction, n_exp, 0, top, 1, 1, 1.f, logits, idx, wt, ws);
+}
+
+int ggb_op_moe_route_softmax_groups(int dt, const void *h, int64_t W, int64_t T, const float *w_router, const float *correction, int n_exp, int n_extra,
+                                    int top, int n_groups, int keep, float scale, float *logits, int32_t *idx, float *wt, int32_t *ws) {
     GGB_REQUIRE_INIT();
     GGB_CHECK_DT(dt);
-    GGB_CHECK_ARG(h && w_router && idx && wt && logits && W > 0 && T > 0 && n_exp > 0 && top > 0 && top <= n_exp && n_exp <= 4096,
+    GGB_CHECK_ARG(h && w_router && idx && wt && logits && W > 0 && T > 0 && n_exp > 0 && n_extra >= 0 && top > 0 && top <= n_exp && n_exp <= 4096,
                   "moe_route_softmax: bad arguments (%d of %d experts)", top, n_exp);
-    const size_t smem = (size_t)(2 * n_exp) * 4;
-    if (T <= 32) { // a step: one launch, and the slot lists of the mat-vec form with it
+    GGB_CHECK_ARG(n_groups > 0 && n_exp % n_groups == 0 && keep > 0 && keep <= n_groups && top <= keep * (n_exp / n_groups),
+                  "moe_route_softmax: %d experts in %d groups of which %d stay cannot give %d experts", n_exp, n_groups, keep, top);
+    const size_t smem = (size_t)(2 * n_exp + n_groups) * 4;
+    const int ldz = n_exp + n_extra;
+    if (T <= kRouteStepTokens) { // a step: one launch, and the slot lists of the mat-vec form with it
         const int64_t n = T * top;
         const int mt = ggb_moe_max_tiles(n, n_exp);
         const bool lists = ws && ggb_moe_step_form(n);
         int32_t *row_src = lists ? ws + n_exp + 1 : nullptr, *inv = lists ? row_src + n : nullptr, *row_expert = lists ? inv + n + 2 * mt + 1 : nullptr;
+        const dim3 grid((unsigned)T, (unsigned)((ldz + kRouteStepWarps - 1) / kRouteStepWarps));
         if (dt == GGB_TYPE_BF16)
-            moe_route_sigmoid_step_kernel<__nv_bfloat16, true><<<dim3((unsigned)T, (unsigned)((n_exp + kRouteStepWarps - 1) / kRouteStepWarps)), 32 * kRouteStepWarps, smem, ggb_cuda_stream()>>>(
-                (const __nv_bfloat16 *)h, W, w_router, correction, n_exp, top, 1, 1, logits, idx, wt, row_src, inv, row_expert);
+            moe_route_sigmoid_step_kernel<__nv_bfloat16, true><<<grid, 32 * kRouteStepWarps, smem, ggb_cuda_stream()>>>(
+                (const __nv_bfloat16 *)h, W, w_router, correction, n_exp, n_extra, top, n_groups, keep, scale, logits, idx, wt, row_src, inv, row_expert);
         else
-            moe_route_sigmoid_step_kernel<float, true><<<dim3((unsigned)T, (unsigned)((n_exp + kRouteStepWarps - 1) / kRouteStepWarps)), 32 * kRouteStepWarps, smem, ggb_cuda_stream()>>>(
-                (const float *)h, W, w_router, correction, n_exp, top, 1, 1, logits, idx, wt, row_src, inv, row_expert);
+            moe_route_sigmoid_step_kernel<float, true><<<grid, 32 * kRouteStepWarps, smem, ggb_cuda_stream()>>>(
+                (const float *)h, W, w_router, correction, n_exp, n_extra, top, n_groups, keep, scale, logits, idx, wt, row_src, inv, row_expert);
         GGB_LAUNCH_CHECK();
         return GGB_OK;
     }
-    const unsigned blocks = (unsigned)((T * n_exp + 7) / 8);
+    const unsigned blocks = (unsigned)((T * ldz + 7) / 8);
     if (dt == GGB_TYPE_BF16)
-        moe_logits_kernel<<<blocks, 256, 0, ggb_cuda_stream()>>>((const __nv_bfloat16 *)h, W, T, w_router, nullptr, n_exp, logits);
+        moe_logits_kernel<<<blocks, 256, 0, ggb_cuda_stream()>>>((const __nv_bfloat16 *)h, W, T, w_router, nullptr, ldz, logits);
     else
-        moe_logits_kernel<<<blocks, 256, 0, ggb_cuda_stream()>>>((const float *)h, W, T, w_router, nullptr, n_exp, logits);
+        moe_logits_kernel<<<blocks, 256, 0, ggb_cuda_stream()>>>((const float *)h, W, T, w_router, nullptr, ldz, logits);
     GGB_LAUNCH_CHECK();
-    moe_select_softmax_kernel<<<(unsigned)T, 32, smem, ggb_cuda_stream()>>>(logits, correction, n_exp, top, idx, wt);
+    moe_select_softmax_kernel<<<(unsigned)T, 32, smem, ggb_cuda_stream()>>>(logits, ldz, correction, n_exp, top, n_groups, keep, scale, idx, wt);
     GGB_LAUNCH_CHECK();
     return GGB_OK;
 }
@@ -501,10 +579,10 @@ int ggb_op_moe_linear_identity(int dt, const void *w, int64_t N, int64_t K, cons
                                int n_identity, const int32_t *ws, int act, float limit, float alpha, void *c, int64_t ldc) {
     GGB_REQUIRE_INIT();
     GGB_CHECK_DT(dt);
-    GGB_CHECK_ARG(w && a && ws && c && N > 0 && K > 0 && T > 0 && lda >= K && ldc >= N && act >= 0 && act <= 3 && n_identity >= 0 &&
+    GGB_CHECK_ARG(w && a && ws && c && N > 0 && K > 0 && T > 0 && lda >= K && ldc >= N && act >= 0 && act <= GGB_ACT_GELU_ERF && n_identity >= 0 &&
                       n_identity < n_exp,
                   "moe_linear: bad arguments");
-    GGB_CHECK_ARG(act < 2 || ggb_moe_step_form(T * top), "moe_linear: the gated forms are built for steps of at most 16 slots");
+    GGB_CHECK_ARG((act != 2 && act != 3) || ggb_moe_step_form(T * top), "moe_linear: the gated forms are built for steps of at most 16 slots");
     const int n_real = n_exp - n_identity;
     const ggb_moe_groups g = groups_of(const_cast<int32_t *>(ws), T * top, n_exp, gather != 0);
     if (ggb_moe_step_form(T * top)) { // decode: every slot is a mat-vec on its expert's matrix
@@ -513,7 +591,8 @@ int ggb_op_moe_linear_identity(int dt, const void *w, int64_t N, int64_t K, cons
         const int32_t *row_expert = g.n_tiles + 1;
         const dim3 grid((unsigned)((N + 7) / 8), (unsigned)(T * top));
 #define MV(E)                                                                                                                         \
-    if (act == 3) moe_vec_kernel<E, 3><<<grid, 256, 0, ggb_cuda_stream()>>>((const E *)w, N, K, (const E *)a, lda, g.row_src, row_expert, nullptr, (E *)c, ldc, vec, n_real, limit, alpha); \
+    if (act == GGB_ACT_GELU_ERF) moe_vec_kernel<E, GGB_ACT_GELU_ERF><<<grid, 256, 0, ggb_cuda_stream()>>>((const E *)w, N, K, (const E *)a, lda, g.row_src, row_expert, nullptr, (E *)c, ldc, vec, n_real, 0.f, 0.f); \
+    else if (act == 3) moe_vec_kernel<E, 3><<<grid, 256, 0, ggb_cuda_stream()>>>((const E *)w, N, K, (const E *)a, lda, g.row_src, row_expert, nullptr, (E *)c, ldc, vec, n_real, limit, alpha); \
     else if (act == 2) moe_vec_kernel<E, 2><<<grid, 256, 0, ggb_cuda_stream()>>>((const E *)w, N, K, (const E *)a, lda, g.row_src, row_expert, nullptr, (E *)c, ldc, vec, n_real, 0.f, 0.f); \
     else if (act) moe_vec_kernel<E, 1><<<grid, 256, 0, ggb_cuda_stream()>>>((const E *)w, N, K, (const E *)a, lda, g.row_src, row_expert, nullptr, (E *)c, ldc, vec, n_real, 0.f, 0.f); \
     else moe_vec_kernel<E, 0><<<grid, 256, 0, ggb_cuda_stream()>>>((const E *)w, N, K, (const E *)a, lda, g.row_src, row_expert, (float *)c, nullptr, ldc, vec, n_real, 0.f, 0.f);
@@ -540,10 +619,44 @@ int ggb_op_moe_linear_identity(int dt, const void *w, int64_t N, int64_t K, cons
             GGB_LAUNCH_CHECK();
             a_sorted = gbuf;
         }
-        return ggb_gemm_grouped_bf16(w, N, K, a_sorted, n, n_real, g.offsets, act ? nullptr : (float *)c, act ? c : nullptr, ldc);
+        return ggb_gemm_grouped_bf16(w, N, K, a_sorted, n, n_real, g.offsets, act ? nullptr : (float *)c, act ? c : nullptr, act, ldc);
     }
     return ggb_linear_grouped_launch(dt, w, N, K, a, lda, ggb_moe_max_tiles(T * top, n_exp), act ? nullptr : (float *)c, act ? c : nullptr,
                                      ldc, act, g);
+}
+
+int ggb_op_moe_linear_shared(int dt, const void *w, int64_t N, int64_t K, const void *a, int64_t lda, int gather, int64_t T, int top, int n_exp,
+                             const int32_t *ws, int act, void *c, int64_t ldc, const void *w_s, int64_t N_s, int64_t K_s, const void *a_s, int64_t lda_s,
+                             void *c_s) {
+    GGB_REQUIRE_INIT();
+    GGB_CHECK_DT(dt);
+    GGB_CHECK_ARG(w && a && ws && c && w_s && a_s && c_s && N > 0 && K > 0 && N_s > 0 && K_s > 0 && T > 0 && lda >= K && ldc >= N && lda_s >= K_s,
+                  "moe_linear_shared: bad arguments");
+    GGB_CHECK_ARG(act == GGB_ACT_NONE || act == GGB_ACT_GELU_ERF, "moe_linear_shared: activation %d", act);
+    if (!ggb_moe_step_form(T * top)) { // portions: the grouped product, then the shared expert's
+        const int rc = ggb_op_moe_linear(dt, w, N, K, a, lda, gather, T, top, n_exp, ws, act, c, ldc);
+        if (rc) return rc;
+        return act ? ggb_op_linear_act(dt, w_s, N_s, K_s, a_s, lda_s, T, act, c_s) : ggb_op_linear(dt, w_s, N_s, K_s, a_s, lda_s, T, (float *)c_s, N_s);
+    }
+    const ggb_moe_groups g = groups_of(const_cast<int32_t *>(ws), T * top, n_exp, gather != 0);
+    const int32_t *row_expert = g.n_tiles + 1;
+    const int ve = 16 / (dt == GGB_TYPE_BF16 ? 2 : 4);
+    const int vec = K % ve == 0 && lda % ve == 0 && ((uintptr_t)w | (uintptr_t)a) % 16 == 0;
+    const int vec_s = K_s % ve == 0 && lda_s % ve == 0 && ((uintptr_t)w_s | (uintptr_t)a_s) % 16 == 0;
+    const dim3 grid((unsigned)((std::max(N, N_s) + 7) / 8), (unsigned)(T * top + T));
+#define MVS(E, ACT)                                                                                                                             \
+    moe_vec_shared_kernel<E, ACT><<<grid, 256, 0, ggb_cuda_stream()>>>((const E *)w, N, K, (const E *)a, lda, g.row_src, row_expert,               \
+                                                                       ACT ? nullptr : (float *)c, ACT ? (E *)c : nullptr, ldc, vec, (int)(T * top), \
+                                                                       shared_product<E>{(const E *)w_s, (const E *)a_s, N_s, K_s, lda_s, N_s,      \
+                                                                                         ACT ? nullptr : (float *)c_s, ACT ? (E *)c_s : nullptr, vec_s});
+    if (dt == GGB_TYPE_BF16) {
+        if (act) MVS(__nv_bfloat16, GGB_ACT_GELU_ERF) else MVS(__nv_bfloat16, GGB_ACT_NONE)
+    } else {
+        if (act) MVS(float, GGB_ACT_GELU_ERF) else MVS(float, GGB_ACT_NONE)
+    }
+#undef MVS
+    GGB_LAUNCH_CHECK();
+    return GGB_OK;
 }
 
 int ggb_op_moe_combine_norm(int dt, const float *y, const int32_t *ws, const float *wt, int64_t T, int top, int n_exp, int64_t W, const float *wa,

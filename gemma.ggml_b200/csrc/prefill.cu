@@ -111,7 +111,8 @@ struct GemmArgs {
     // grouped form (mixture of experts, plain bf16 matrices): blockIdx.z = expert e, whose matrix is seg[0].qs + e * rows * K
     // and whose rows of A / C are [m_ranges[e], m_ranges[e + 1]) (device int32); tiles past the range leave at once
     const int32_t *m_ranges;
-    __nv_bfloat16 *act_out; // when set: C is stored as bf16 relu(c)^2 with row pitch seg[0].ldc instead of fp32
+    __nv_bfloat16 *act_out; // when set: C is stored as bf16 act(c) (GGB_ACT_*) with row pitch seg[0].ldc instead of fp32
+    int act;
 };
 
 // int8 / int4 code -> fp32 without the conversion pipe: the (biased) code is dropped into the mantissa of
@@ -323,15 +324,14 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16w_kernel(const GemmA
             for (int c0 = chalf * (BN / 4); c0 < (chalf + 1) * (BN / 4); c0 += 32) {
                 uint32_t v[32];
                 tmem_ld32(tmem_base + ((uint32_t)(lq * 32) << 16) + (uint32_t)(mt * BN + c0), v);
-                if (row < m_end && sn0 + c0 < sg.rows && A.act_out) { // expert activation: relu(c)^2 as bf16
+                if (row < m_end && sn0 + c0 < sg.rows && A.act_out && !A.ws) { // the next product's operand
                     __nv_bfloat16 *dst = A.act_out + (size_t)row * sg.ldc + sn0 + c0;
 #pragma unroll
                     for (int u = 0; u < 32; u += 8) {
                         __align__(16) __nv_bfloat16 o[8];
 #pragma unroll
                         for (int q = 0; q < 8; q++) {
-                            const float f = __uint_as_float(v[u + q]);
-                            o[q] = __float2bfloat16_rn(f > 0.f ? f * f : 0.f);
+                            o[q] = __float2bfloat16_rn(act_f32(__uint_as_float(v[u + q]), A.act));
                         }
                         *reinterpret_cast<uint4 *>(dst + u) = *reinterpret_cast<const uint4 *>(o);
                     }
@@ -404,7 +404,8 @@ __global__ void splitk_reduce_kernel(const GemmArgs A, int splits) {
     float acc = A.ws[i];
     for (int s = 1; s < splits; s++) acc += A.ws[(int64_t)s * T * N + i];
     if (A.resid) acc += A.resid[t * sg.ldc + col];
-    sg.c[t * sg.ldc + col] = acc;
+    if (A.act_out) A.act_out[t * sg.ldc + col] = __float2bfloat16_rn(act_f32(acc, A.act));
+    else sg.c[t * sg.ldc + col] = acc;
 }
 
 // rms_norm * w -> bf16 (the A operand of the next GEMM): same double-sum order as rms_norm_kernel (elementwise.cu)
@@ -766,17 +767,18 @@ int ggb_op_geglu_bf16(const float *gate, const float *up, int64_t n, void *y_bf1
 }
 
 static int gemm_launch(int n, const ggb_weight *const *w, const void *a_bf16, int64_t T, float *const *c, const int64_t *ldc,
-                       const float *resid, void *workspace, size_t workspace_bytes) {
+                       const float *resid, void *workspace, size_t workspace_bytes, void *act_out = nullptr, int act = 0) {
     GGB_REQUIRE_INIT();
     GGB_CHECK_ARG(n >= 1 && n <= kMaxSegs && w && a_bf16 && c && ldc && T > 0, "bad gemm args");
-    GGB_CHECK_ARG(n == 1 || !resid, "gemm: a residual needs a single matrix");
+    GGB_CHECK_ARG(n == 1 || (!resid && !act_out), "gemm: a residual or an activation needs a single matrix");
+    GGB_CHECK_ARG(!act_out || (!resid && ldc[0] % 8 == 0), "gemm: an activation takes no residual and rows of whole 16-byte pieces");
     const int64_t K = w[0]->cols;
     const int type = w[0]->type;
     GGB_CHECK_ARG(type == GGB_TYPE_Q4_0 || type == GGB_TYPE_Q8_0 || type == GGB_TYPE_BF16, "gemm: weight type %d", type);
     GemmArgs A{};
     int64_t N = 0;
     for (int i = 0; i < n; i++) {
-        GGB_CHECK_ARG(w[i] && c[i] && w[i]->cols == K && w[i]->type == type, "gemm: matrices of one launch share K and the type");
+        GGB_CHECK_ARG(w[i] && (c[i] || act_out) && w[i]->cols == K && w[i]->type == type, "gemm: matrices of one launch share K and the type");
         const int64_t rows = w[i]->rows;
         GGB_CHECK_ARG(K % 64 == 0 && rows % 32 == 0 && ldc[i] >= rows && ldc[i] % 4 == 0,
                       "gemm needs K %% 64 == 0, N %% 32 == 0 (N=%lld K=%lld)", (long long)rows, (long long)K);
@@ -802,6 +804,8 @@ static int gemm_launch(int n, const ggb_weight *const *w, const void *a_bf16, in
     A.kblocks_per_split = (kblocks + splits - 1) / splits;
     A.ws = splits > 1 ? (float *)workspace : nullptr;
     A.resid = resid;
+    A.act_out = (__nv_bfloat16 *)act_out;
+    A.act = act;
     const dim3 grid((unsigned)n_tiles, (unsigned)m_tiles, (unsigned)splits);
     if (splits > 1) A.resid = nullptr; // added by the reducer
     if (type == GGB_TYPE_Q4_0) gemm_bf16w_kernel<GGB_TYPE_Q4_0><<<grid, kGemmThreads, kGemmSmem, ggb_cuda_stream()>>>(A);
@@ -871,7 +875,7 @@ int ggb_op_attn_prefill(const float *q, const void *kcache, const void *vcache, 
 // the rows of expert e (device).  One launch: grid (N tiles, row tiles of the longest possible group, experts).
 bool ggb_gemm_grouped_bf16_fits(int64_t N, int64_t K, int64_t ldc) { return K % 64 == 0 && N % 32 == 0 && ldc % 8 == 0; }
 int ggb_gemm_grouped_bf16(const void *w, int64_t N, int64_t K, const void *a, int64_t n_rows, int n_exp, const int32_t *offsets, float *c,
-                          void *c_act, int64_t ldc) {
+                          void *c_act, int act, int64_t ldc) {
     GGB_REQUIRE_INIT();
     static bool attr_done = false;
     if (!attr_done) {
@@ -886,6 +890,7 @@ int ggb_gemm_grouped_bf16(const void *w, int64_t N, int64_t K, const void *a, in
     A.kblocks_per_split = (int)(K / BK);
     A.m_ranges = offsets;
     A.act_out = (__nv_bfloat16 *)c_act;
+    A.act = act;
     const dim3 grid((unsigned)((N + BN - 1) / BN), (unsigned)((n_rows + BM - 1) / BM), (unsigned)n_exp);
     gemm_bf16w_kernel<GGB_TYPE_BF16><<<grid, kGemmThreads, kGemmSmem, ggb_cuda_stream()>>>(A);
     GGB_LAUNCH_CHECK();
@@ -898,7 +903,7 @@ int ggb_gemm_grouped_bf16(const void *w, int64_t N, int64_t K, const void *a, in
 bool ggb_gemm_dense_bf16_fits(int64_t N, int64_t K, int64_t T, int64_t ldc) {
     return T >= 64 && K % 64 == 0 && N % 32 == 0 && ldc % 4 == 0 && N < (1ll << 31) && K < (1ll << 31) && T < (1ll << 31);
 }
-int ggb_gemm_dense_bf16(const void *w, int64_t N, int64_t K, const void *a, int64_t T, float *c, int64_t ldc) {
+int ggb_gemm_dense_bf16(const void *w, int64_t N, int64_t K, const void *a, int64_t T, float *c, int64_t ldc, void *c_act, int act) {
     GGB_REQUIRE_INIT();
     static void *ws = nullptr;
     static size_t ws_bytes = 0;
@@ -919,5 +924,5 @@ int ggb_gemm_dense_bf16(const void *w, int64_t N, int64_t K, const void *a, int6
     const ggb_weight *wp[1] = {&wd};
     float *cs[1] = {c};
     const int64_t ls[1] = {ldc};
-    return gemm_launch(1, wp, a, T, cs, ls, nullptr, ws, ws_bytes);
+    return gemm_launch(1, wp, a, T, cs, ls, nullptr, ws, ws_bytes, c_act, act);
 }

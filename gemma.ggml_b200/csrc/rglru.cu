@@ -381,7 +381,7 @@ int ggb_op_rglru_gates(int dt, const float *u, const void *split, const int32_t 
     GGB_CHECK_ARG(u && w_ri && z && T > 0 && nb > 0 && d > 0 && nb <= 65535, "rglru_gates: bad arguments");
     if (split && w_ri3 && ggb_rglru_split_fits(dt, T, d)) { // every block is a group of T rows of its own
         GGB_CHECK_ARG(offsets != nullptr, "rglru_gates: the split form needs its offsets");
-        return ggb_gemm_grouped_bf16(w_ri3, 2 * (int64_t)d, 3 * (int64_t)d, split, T, nb, offsets, z, nullptr, 2 * (int64_t)d);
+        return ggb_gemm_grouped_bf16(w_ri3, 2 * (int64_t)d, 3 * (int64_t)d, split, T, nb, offsets, z, nullptr, GGB_ACT_NONE, 2 * (int64_t)d);
     }
     const dim3 grid((unsigned)((2 * d + 63) / 64), (unsigned)((T + 63) / 64), (unsigned)nb);
     if (dt == GGB_TYPE_BF16) rglru_gates_kernel<<<grid, 256, 0, ggb_cuda_stream()>>>(u, T, nb, d, (const __nv_bfloat16 *)w_ri, z);

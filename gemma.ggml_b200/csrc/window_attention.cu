@@ -25,6 +25,9 @@
 // both maps of a head, so every value row is read once for both, and the combination is the epilogue of the kernel that
 // holds the sums.
 //
+// One-map heads have two more choices at their end: a sink per head (one more exp(sink) in the soft-max's denominator that no
+// value goes with) and the gate per element.  head_qkv_store divides every head of q and k by its own root mean square.
+//
 // Compiled with -fmad=false: multiply-adds are spelled fmaf().
 #include <algorithm>
 
@@ -37,12 +40,13 @@ constexpr int kMaxDvRegs = 8; // value coordinates per lane: Dv <= 32 * kMaxDvRe
 constexpr int kWarps = 8;
 constexpr int kMaxSplit = 16; // CTAs that share one (token, head) of a short step
 
-// what MAPS 2 does with the two weighted sums of a head: o = a1 - lambda a2; o <- o / sqrt(mean(o^2) + eps) * scale *
-// sigmoid(gate[token][head * Dv + c])
-struct diff_args {
+// what becomes of a head's weighted sums.  MAPS 1: the sum over l, or over l + exp(sink[head]) with a sink.  MAPS 2: o = a1 -
+// lambda a2; o <- o / sqrt(mean(o^2) + eps) * scale.  Then, with a gate, times sigmoid(gate[token][head * Dv + c])
+struct finish_args {
     float lambda = 0.f, scale = 1.f, eps = 0.f;
     const float *gate = nullptr; // fp32 rows of stride ldg, or null
     int64_t ldg = 0;
+    const float *sink = nullptr; // a score per head, or null
 };
 
 // the first position the query at position i sees: everything (size <= 0), the last `size` positions, or its chunk
@@ -136,16 +140,65 @@ __global__ void __launch_bounds__(256) window_qkv_store_kernel(const float *__re
     }
 }
 
+// the same with a norm per head: a warp takes one head of q, k or v of one token (rows y * 8 + warp of H + 2 G).  q and k are divided
+// by the root mean square over the head's D numbers, times a weight of D numbers that all heads share (null: none), before the rotation.
+template <typename E>
+__global__ void __launch_bounds__(256) head_qkv_store_kernel(const float *__restrict__ q, const float *__restrict__ k, const float *__restrict__ v, int64_t ld,
+                                                             int H, int G, int D, int Dv, const float *__restrict__ qn_w, const float *__restrict__ kn_w,
+                                                             float eps, int rot_dims, int rot_halves, const float *__restrict__ cs, float scale,
+                                                             const int32_t *__restrict__ pos0, const int32_t *__restrict__ table, int B,
+                                                             E *__restrict__ cache, int64_t cache_ld, float *__restrict__ q_out) {
+    const int lane = threadIdx.x & 31, item = (int)blockIdx.y * 8 + (int)(threadIdx.x >> 5);
+    if (item >= H + 2 * G) return;
+    const int64_t t = blockIdx.x, pos = (int64_t)*pos0 + t;
+    E *row = cache + ((int64_t)table[pos / B] * B + pos % B) * cache_ld;
+    if (item >= H + G) { // a value head
+        const int g = item - H - G;
+        const float *src = v + t * ld + (int64_t)g * Dv;
+        E *dst = row + (int64_t)G * D + (int64_t)g * Dv;
+        for (int c = lane; c < Dv; c += 32) dst[c] = from_f32<E>(src[c]);
+        return;
+    }
+    const bool is_q = item < H;
+    const float *src = is_q ? q + t * ld + (int64_t)item * D : k + t * ld + (int64_t)(item - H) * D;
+    const float *nw = is_q ? qn_w : kn_w;
+    float ss = 0.f;
+    for (int d = lane; d < D; d += 32) ss = fmaf(src[d], src[d], ss);
+    const float r = 1.0f / sqrtf(warp_sum_f32(ss) / (float)D + eps);
+    float *qd = q_out + (t * H + item) * D;
+    E *kd = row + (int64_t)(item - H) * D;
+    auto normed = [&](int d) { return nw ? src[d] * r * nw[d] : src[d] * r; };
+    auto put = [&](int d, float x) {
+        if (is_q) qd[d] = x * scale;
+        else kd[d] = from_f32<E>(x);
+    };
+    const int half = rot_dims / 2;
+    const float *ct = cs + pos * rot_dims;
+    for (int m = lane; m < half; m += 32) {
+        const int d0 = rot_halves ? m : 2 * m, d1 = rot_halves ? m + half : 2 * m + 1;
+        const float u = normed(d0), w = normed(d1), c = ct[2 * m], s = ct[2 * m + 1];
+        put(d0, u * c - w * s);
+        put(d1, w * c + u * s);
+    }
+    for (int d = rot_dims + lane; d < D; d += 32) put(d, normed(d));
+}
+
 template <typename E> struct RowVec { // 16 bytes of a cache row
     static constexpr int n = 16 / (int)sizeof(E);
     uint4 raw;
     __device__ __forceinline__ float at(int i) const { return to_f32(reinterpret_cast<const E *>(&raw)[i]); }
 };
 
-// what a head's weighted sum becomes: divided by the soft-max sum, turned back by the reader's position, stored
+// what a head's weighted sum becomes: divided by the soft-max sum, turned back by the reader's position, gated, stored
 template <typename E, int NP = kMaxDvRegs / 2>
-__device__ __forceinline__ void window_finish(const float *acc, float l, int64_t i, int lane, int Dv, const float *__restrict__ cs_v, E *orow) {
-    const float inv = 1.0f / l;
+__device__ __forceinline__ void window_finish(const float *acc, float m, float l, int64_t i, int64_t t, int h, int lane, int Dv,
+                                              const float *__restrict__ cs_v, const finish_args &fa, E *orow) {
+    float inv = 1.0f / l;
+    if (fa.sink) { // sum and weighted sum are relative to the running maximum m (finite: a query sees itself)
+        const float s0 = fa.sink[h], M = fmaxf(m, s0), f = expf(m - M);
+        inv = f / (l * f + expf(s0 - M));
+    }
+    const float *gr = fa.gate ? fa.gate + t * fa.ldg + (int64_t)h * Dv : nullptr;
     const float *cv = cs_v ? cs_v + i * (Dv / 2) * 2 : nullptr;
 #pragma unroll
     for (int r = 0; r < NP; r++) {
@@ -158,6 +211,10 @@ __device__ __forceinline__ void window_finish(const float *acc, float l, int64_t
                 u = u2;
                 w = w2;
             }
+            if (gr) {
+                u = u / (1.0f + expf(-gr[c]));
+                w = w / (1.0f + expf(-gr[c + 1]));
+            }
             orow[c] = from_f32<E>(u);
             orow[c + 1] = from_f32<E>(w);
         }
@@ -167,7 +224,7 @@ __device__ __forceinline__ void window_finish(const float *acc, float l, int64_t
 // the same for the two maps of a differential head (all lanes of the warp take part)
 template <typename E, int NP = kMaxDvRegs / 2>
 __device__ __forceinline__ void diff_finish(const float *acc1, float l1, const float *acc2, float l2, int64_t t, int h, int lane, int Dv,
-                                            const diff_args &da, E *orow) {
+                                            const finish_args &da, E *orow) {
     const float i1 = 1.0f / l1, i2 = da.lambda / l2;
     float o[2 * NP], ss = 0.f;
 #pragma unroll
@@ -214,7 +271,7 @@ template <typename E, int MAPS>
 __global__ void __launch_bounds__(32 * kWarps) window_attn_kernel(const float *__restrict__ q, const E *__restrict__ cache, int64_t cache_ld,
                                                                   const int32_t *__restrict__ table, int B, const int32_t *__restrict__ pos0,
                                                                   int64_t T, int H, int G, int D, int Dv, int64_t window, int chunked, int64_t keep,
-                                                                  float cap, const float *__restrict__ cs_v, diff_args da, E *__restrict__ out,
+                                                                  float cap, const float *__restrict__ cs_v, finish_args da, E *__restrict__ out,
                                                                   int vec, float *__restrict__ part_out) {
     extern __shared__ __align__(16) float wa_smem[]; // q: [kWarps][MAPS][Dp]; merge: [kWarps][MAPS][kPartW]
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -374,24 +431,25 @@ __global__ void __launch_bounds__(32 * kWarps) window_attn_kernel(const float *_
         return;
     }
     E *orow = out + (t * H + h) * Dv;
-    if (MAPS == 1) window_finish(acc[0], l[0], i, lane, Dv, cs_v, orow);
+    if (MAPS == 1) window_finish(acc[0], m[0], l[0], i, t, h, lane, Dv, cs_v, da, orow);
     else diff_finish(acc[0], l[0], acc[MAPS - 1], l[MAPS - 1], t, h, lane, Dv, da, orow);
 }
 
 // one warp per (token, head): the splits' parts merged, then as above
 template <typename E, int MAPS>
 __global__ void __launch_bounds__(32) window_merge_kernel(const float *__restrict__ part, int n_split, const int32_t *__restrict__ pos0, int H, int Dv,
-                                                         const float *__restrict__ cs_v, diff_args da, E *__restrict__ out) {
+                                                         const float *__restrict__ cs_v, finish_args da, E *__restrict__ out) {
     const int64_t t = blockIdx.x;
     const int h = blockIdx.y, lane = threadIdx.x;
     constexpr int pw = MAPS * kPartW;
-    float l[MAPS], acc[MAPS][kMaxDvRegs];
+    float m[MAPS], l[MAPS], acc[MAPS][kMaxDvRegs];
 #pragma unroll
     for (int a = 0; a < MAPS; a++) {
         const float *pp = part + (t * H + h) * n_split * pw + a * kPartW;
         float M = -INFINITY;
 #pragma unroll 4
         for (int s = 0; s < n_split; s++) M = fmaxf(M, pp[s * pw]);
+        m[a] = M;
         l[a] = 0.f;
 #pragma unroll
         for (int r = 0; r < kMaxDvRegs; r++) acc[a][r] = 0.f;
@@ -404,7 +462,7 @@ __global__ void __launch_bounds__(32) window_merge_kernel(const float *__restric
         }
     }
     E *orow = out + (t * H + h) * Dv;
-    if (MAPS == 1) window_finish(acc[0], l[0], (int64_t)*pos0 + t, lane, Dv, cs_v, orow);
+    if (MAPS == 1) window_finish(acc[0], m[0], l[0], (int64_t)*pos0 + t, t, h, lane, Dv, cs_v, da, orow);
     else diff_finish(acc[0], l[0], acc[MAPS - 1], l[MAPS - 1], t, h, lane, Dv, da, orow);
 }
 
@@ -420,7 +478,7 @@ __global__ void __launch_bounds__(32 * kWarps) window_attn_tile_kernel(const flo
                                                                        const int32_t *__restrict__ table, int B, const int32_t *__restrict__ pos0,
                                                                        int64_t T, int H, int G, int D, int Dv, int kp, int vp, int64_t window,
                                                                        int chunked, int64_t keep, float cap, const float *__restrict__ cs_v,
-                                                                       diff_args da, E *__restrict__ out) {
+                                                                       finish_args da, E *__restrict__ out) {
     extern __shared__ __align__(16) float wa_smem[];
     const int Dp = (D + 3) & ~3;
     float *sq = wa_smem;               // [kQT][MAPS][Dp]
@@ -568,7 +626,7 @@ __global__ void __launch_bounds__(32 * kWarps) window_attn_tile_kernel(const flo
         const int qi = warp * kQPW + a;
         if (qi >= nq) continue;
         E *orow = out + ((t0 + qi) * H + h) * Dv;
-        if (MAPS == 1) window_finish<E, NP>(acc[a][0], l[a][0], i0 + qi, lane, Dv, cs_v, orow);
+        if (MAPS == 1) window_finish<E, NP>(acc[a][0], m[a][0], l[a][0], i0 + qi, t0 + qi, h, lane, Dv, cs_v, da, orow);
         else diff_finish<E, NP>(acc[a][0], l[a][0], acc[a][MAPS - 1], l[a][MAPS - 1], t0 + qi, h, lane, Dv, da, orow);
     }
 }
@@ -617,6 +675,26 @@ int ggb_op_masked_qkv_store(int dt, const float *q, const float *k, const float 
                             block_size, ggb_window_cache_ld(G, D, Dv), cache, q_out);
 }
 
+int ggb_op_head_qkv_store(int dt, const float *q, const float *k, const float *v, int64_t ld, int64_t T, int H, int G, int D, int Dv, const float *qn_w,
+                          const float *kn_w, float eps, int rot_dims, int rot_halves, const float *cos_sin, float scale, const int32_t *pos0,
+                          const int32_t *block_table, int block_size, void *cache, float *q_out) {
+    GGB_REQUIRE_INIT();
+    GGB_CHECK_ARG(dt == GGB_TYPE_BF16 || dt == GGB_TYPE_F32, "head_qkv_store: dtype %d is neither bf16 nor f32", dt);
+    GGB_CHECK_ARG(q && k && v && pos0 && block_table && cache && q_out && T > 0 && H > 0 && G > 0 && H % G == 0 && block_size > 0 && D > 0 && Dv > 0,
+                  "head_qkv_store: bad arguments");
+    GGB_CHECK_ARG(rot_dims >= 0 && rot_dims <= D && rot_dims % 2 == 0 && (!rot_dims || cos_sin), "head_qkv_store: %d of %d dimensions cannot turn", rot_dims, D);
+    const int64_t cld = ggb_window_cache_ld(G, D, Dv);
+    const dim3 grid((unsigned)T, (unsigned)((H + 2 * G + 7) / 8));
+    if (dt == GGB_TYPE_BF16)
+        head_qkv_store_kernel<<<grid, 256, 0, ggb_cuda_stream()>>>(q, k, v, ld, H, G, D, Dv, qn_w, kn_w, eps, rot_dims, rot_halves, cos_sin, scale, pos0,
+                                                                   block_table, block_size, (__nv_bfloat16 *)cache, cld, q_out);
+    else
+        head_qkv_store_kernel<<<grid, 256, 0, ggb_cuda_stream()>>>(q, k, v, ld, H, G, D, Dv, qn_w, kn_w, eps, rot_dims, rot_halves, cos_sin, scale, pos0,
+                                                                   block_table, block_size, (float *)cache, cld, q_out);
+    GGB_LAUNCH_CHECK();
+    return GGB_OK;
+}
+
 int ggb_op_diff_qkv_store(int dt, const float *q, const float *k, const float *v, int64_t ld, int64_t T, int H, int G, int D, int Dv, int rot_dims,
                           int rot_halves, const float *cos_sin_k, float scale, const int32_t *pos0, const int32_t *block_table, int block_size,
                           void *cache, float *q_out) {
@@ -636,7 +714,7 @@ int ggb_op_window_attn(int dt, const float *q, const void *cache, const int32_t 
 template <int MAPS>
 static int masked_attn_launch(int dt, const float *q, const void *cache, const int32_t *block_table, int block_size, const int32_t *pos0, int64_t T,
                               int H, int G, int D, int Dv, int64_t window, int chunked, int64_t keep, float softcap, const float *cos_sin_v,
-                              const diff_args &da, void *out, float *scratch) {
+                              const finish_args &da, void *out, float *scratch) {
     GGB_REQUIRE_INIT();
     GGB_CHECK_ARG(softcap >= 0.f && (chunked == 0 || chunked == 1), "masked_attn: the soft cap must not be negative");
     GGB_CHECK_ARG(dt == GGB_TYPE_BF16 || dt == GGB_TYPE_F32, "window_attn: dtype %d is neither bf16 nor f32", dt);
@@ -708,14 +786,23 @@ extern "C" {
 int ggb_op_masked_attn(int dt, const float *q, const void *cache, const int32_t *block_table, int block_size, const int32_t *pos0, int64_t T,
                        int H, int G, int D, int Dv, int64_t window, int chunked, float softcap, const float *cos_sin_v, void *out,
                        float *scratch) {
-    return masked_attn_launch<1>(dt, q, cache, block_table, block_size, pos0, T, H, G, D, Dv, window, chunked, 0, softcap, cos_sin_v, diff_args{}, out,
+    return masked_attn_launch<1>(dt, q, cache, block_table, block_size, pos0, T, H, G, D, Dv, window, chunked, 0, softcap, cos_sin_v, finish_args{}, out,
                                  scratch);
 }
 
 int ggb_op_masked_attn_keep(int dt, const float *q, const void *cache, const int32_t *block_table, int block_size, const int32_t *pos0, int64_t T,
                             int H, int G, int D, int Dv, int64_t window, int64_t keep_first, float softcap, void *out, float *scratch) {
-    return masked_attn_launch<1>(dt, q, cache, block_table, block_size, pos0, T, H, G, D, Dv, window, 0, keep_first, softcap, nullptr, diff_args{}, out,
+    return masked_attn_launch<1>(dt, q, cache, block_table, block_size, pos0, T, H, G, D, Dv, window, 0, keep_first, softcap, nullptr, finish_args{}, out,
                                  scratch);
+}
+
+int ggb_op_masked_attn_gated(int dt, const float *q, const void *cache, const int32_t *block_table, int block_size, const int32_t *pos0, int64_t T,
+                             int H, int G, int D, int Dv, int64_t window, int64_t keep_first, float softcap, const float *sink, const float *gate,
+                             int64_t ldg, void *out, float *scratch) {
+    GGB_CHECK_ARG(!gate || ldg >= (int64_t)H * Dv, "masked_attn_gated: a gate row holds a number per output");
+    finish_args fa;
+    fa.sink = sink, fa.gate = gate, fa.ldg = ldg;
+    return masked_attn_launch<1>(dt, q, cache, block_table, block_size, pos0, T, H, G, D, Dv, window, 0, keep_first, softcap, nullptr, fa, out, scratch);
 }
 
 int ggb_op_diff_attn(int dt, const float *q, const void *cache, const int32_t *block_table, int block_size, const int32_t *pos0, int64_t T, int H,
@@ -723,7 +810,7 @@ int ggb_op_diff_attn(int dt, const float *q, const void *cache, const int32_t *b
                      const float *gate, int64_t ldg, void *out, float *scratch) {
     GGB_CHECK_ARG(!gate || ldg >= (int64_t)H * Dv, "diff_attn: a gate row holds a number per output");
     return masked_attn_launch<2>(dt, q, cache, block_table, block_size, pos0, T, H, G, D, Dv, window, 0, keep_first, softcap, nullptr,
-                                 diff_args{lambda, out_scale, eps, gate, ldg}, out, scratch);
+                                 finish_args{lambda, out_scale, eps, gate, ldg, nullptr}, out, scratch);
 }
 
 } // extern "C"

@@ -11,6 +11,7 @@
 #include "lm_engine.h"
 #include "begupel_model.h"
 #include "ditalorn_model.h"
+#include "fekopel_model.h"
 #include "kibilix_model.h"
 #include "tezesun_model.h"
 #include "safolorn_model.h"
@@ -274,6 +275,24 @@ int tz_config_probe(const char *text, int64_t *out) {
     }
     out[0] = (int64_t)c.layers.size(); out[1] = n[0]; out[2] = n[1]; out[3] = n[2]; out[4] = ff; out[5] = c.vocab; out[6] = c.width;
     tz_lookback(c, &out[7], &out[8]);
+    return 0;
+}
+// host only: reads a Fekopel configuration; fills out[10] = {layers, attention, attention_2, with experts, with a shared expert, vocab,
+// width, layer runs, positions the farthest-looking layer sees (0: all), kept first positions}
+int fk_config_probe(const char *text, int64_t *out) {
+    json_value j;
+    fk_config c;
+    if (!json_parser(text, strlen(text)).parse(&j, &g_capi_err)) return -1;
+    if (fk_parse_config(j, nullptr, &c, &g_capi_err)) return -1;
+    int64_t n[2] = {0, 0}, moe = 0, shared = 0;
+    for (const auto &l : c.layers) {
+        n[l.mix.gated]++;
+        moe += l.moe.experts > 0;
+        shared += l.moe.shared_ff > 0;
+    }
+    const int64_t v[8] = {(int64_t)c.layers.size(), n[0], n[1], moe, shared, c.vocab, c.width, (int64_t)c.runs.size()};
+    std::copy(v, v + 8, out);
+    fk_lookback(c, &out[8], &out[9]);
     return 0;
 }
 // host only: a tensor of a .safetensors file: returns its number of dimensions (shape[0 .. 8) filled, *nbytes, dtype text),

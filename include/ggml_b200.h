@@ -318,9 +318,27 @@ int ggb_op_hyper_mix_moe(int dt, float *xs, const float *y2, const int32_t *ws, 
  * tile kernel with the activation as its epilogue) except for the shapes the tensor cores take, which go through scratch
  * (fp32 [T][N]; NULL: never) and ggb_op_act_rows */
 int ggb_op_linear_relu2(int dt, const void *w, int64_t N, int64_t K, const void *a, int64_t lda, int64_t T, float *scratch, void *y);
-/* y (dt, dense [T][F]) = act(x), x fp32 rows of stride ldx; act 0: as it is, 1: relu(x)^2 */
+/* activations of a product that is not gated (2 and 3 are the gated forms of ggb_op_moe_linear): as it is, relu(z)^2, z times the normal
+ * distribution function at z */
+#define GGB_ACT_NONE 0
+#define GGB_ACT_RELU2 1
+#define GGB_ACT_GELU_ERF 4
+/* y (dt, dense [T][N]) = act(a w^T), the activation as the epilogue of every form of the product (one launch, or the product's own
+ * split and its reduction) */
+int ggb_op_linear_act(int dt, const void *w, int64_t N, int64_t K, const void *a, int64_t lda, int64_t T, int act, void *y);
+/* y (dt, dense [T][F]) = act(x), x fp32 rows of stride ldx; act: GGB_ACT_* */
 int ggb_op_act_rows(int dt, const float *x, int64_t ldx, int64_t T, int64_t F, int act, void *y);
 
+/* The pass between two sublayers with a layer norm (csrc/residual.cu).  x' = x (NULL: zero), + y ([T][W], a sublayer's output) or + a
+ * mixture of experts whose weighted sum has not been taken yet (slot rows y2 with ws, wt, n_exp of ggb_op_moe_group for T_slots tokens, at
+ * most GGB_RESIDUAL_MAX_TOP slots each, and with ys ([T][W]) an expert that every token uses, times sigmoid(gate[t * ldg]) or, with gate
+ * NULL, one), + the tokens' rows of an embedding table (dt; table NULL: none; with x NULL the residual starts as that row), + add ([W], may
+ * be NULL).  x_out (fp32, may be x or NULL) = x'; h (dt, may be NULL) = (x' - mean) / sqrt(mean of (x' - mean)^2 + eps) * nw + nb.
+ * rows (device int32): only the tokens rows[0 .. T), outputs dense in that order. */
+#define GGB_RESIDUAL_MAX_TOP 64
+int ggb_op_residual_layer_norm(int dt, const float *x, const float *y, const float *y2, const int32_t *ws, const float *wt, int64_t T_slots, int top, int n_exp,
+                               const float *ys, const float *gate, int64_t ldg, const void *table, const int32_t *ids, const float *add, const float *nw,
+                               const float *nb, float eps, int64_t W, int64_t T, const int32_t *rows, float *x_out, void *h);
 /* Layers whose two sublayers read one normed input side by side.  One pass between two such layers: x' = x + (a * ls_a +
  * b * ls_b) per channel (a, then b, may be NULL) -> x_out (fp32, another buffer than x, may be NULL); h = x' / sqrt(mean(x'^2) +
  * eps) * nw in dt (nw NULL: none; h may be NULL); with mu the token shift hs = h + (h_before - h) * mu in dt, h_before the row of
@@ -435,6 +453,16 @@ int ggb_op_masked_attn(int dt, const float *q, const void *cache, const int32_t 
 /* a window that keeps the first positions visible: the query at position i sees j <= i with i - j < window or j < keep_first */
 int ggb_op_masked_attn_keep(int dt, const float *q, const void *cache, const int32_t *block_table, int block_size, const int32_t *pos0, int64_t T,
                             int H, int G, int D, int Dv, int64_t window, int64_t keep_first, float softcap, void *out, float *scratch);
+/* the same with a sink per head (fp32 [H] scores, NULL: none): exp(sink[h]) more in the soft-max's denominator, with no value; and / or a
+ * gate: out times sigmoid(gate) per element (fp32 rows of stride ldg, a number per output; NULL: none) */
+int ggb_op_masked_attn_gated(int dt, const float *q, const void *cache, const int32_t *block_table, int block_size, const int32_t *pos0, int64_t T,
+                             int H, int G, int D, int Dv, int64_t window, int64_t keep_first, float softcap, const float *sink, const float *gate,
+                             int64_t ldg, void *out, float *scratch);
+/* ggb_op_masked_qkv_store with a norm per head: every head of q and k is divided by the root of (its mean square + eps), times qn_w /
+ * kn_w (D numbers shared by all heads; NULL: no weight), before the rotation; values are stored as they are */
+int ggb_op_head_qkv_store(int dt, const float *q, const float *k, const float *v, int64_t ld, int64_t T, int H, int G, int D, int Dv, const float *qn_w,
+                          const float *kn_w, float eps, int rot_dims, int rot_halves, const float *cos_sin, float scale, const int32_t *pos0,
+                          const int32_t *block_table, int block_size, void *cache, float *q_out);
 /* Differential attention: every head has two query / key maps over the same values.  q [T][H][2][D], k [T][G][2][D], v
  * [T][G][Dv] raw projections; cache row [k (G * 2 * D) | v (G * Dv)], ggb_window_cache_ld(G, 2 * D, Dv) numbers apart; q_out
  * [T][H][2][D].  Each map is a soft-max attention of its own (window, keep_first, softcap as above); with a1, a2 their outputs
@@ -522,7 +550,7 @@ int ggb_op_latent_attn_out_gated(int dt, const float *part, int n_split, const f
  * route: fp32 logits w_router h + bias, the `top` largest (ties: lower index), weights = soft-max over the chosen.
  * group: sorts the T * top slots by expert into `ws` (ggb_moe_group_ints int32).  moe_linear: per expert
  * c[sorted row] = a[row] w_e^T with w = [n_exp][N][K]; gather: a is indexed by token (first product), else by sorted
- * row; act 1: c = relu(.)^2 in dt, act 0: c fp32.  combine: out[t] = sum_s wt[t][s] y[sorted row of slot s]. */
+ * row; act GGB_ACT_RELU2 or GGB_ACT_GELU_ERF: c = act(.) in dt, act 0: c fp32.  combine: out[t] = sum_s wt[t][s] y[sorted row of slot s]. */
 int ggb_op_moe_route(int dt, const void *h, int64_t W, int64_t T, const float *w_router, const float *bias, int n_exp, int top,
                      float *logits /* scratch [T][n_exp] */, int32_t *idx, float *wt);
 /* route with sigmoid scores: s = sigmoid(w_router h) in fp32; the choice score of an expert is s + correction (may be
@@ -552,6 +580,18 @@ int ggb_op_moe_combine_norm(int dt, const float *y, const int32_t *ws, const flo
  * ggb_op_moe_route_sigmoid. */
 int ggb_op_moe_route_softmax(int dt, const void *h, int64_t W, int64_t T, const float *w_router, const float *correction, int n_exp, int top,
                              float *logits /* scratch [T][n_exp] */, int32_t *idx, float *wt, int32_t *ws);
+/* the same with groups, a factor and more rows: the experts form n_groups equal groups of neighbours, a group's score is its largest
+ * s + correction, and only experts of the `keep` best groups can be chosen; the weights are times `scale`.  w_router may have n_extra
+ * more rows behind the experts' (a gate that reads the same input, say): logits is [T][n_exp + n_extra] and holds their products
+ * behind the experts' logits. */
+int ggb_op_moe_route_softmax_groups(int dt, const void *h, int64_t W, int64_t T, const float *w_router, const float *correction, int n_exp, int n_extra,
+                                    int top, int n_groups, int keep, float scale, float *logits, int32_t *idx, float *wt, int32_t *ws);
+/* moe_linear and, beside it, the same product of an expert that every token uses, whose matrix w_s [N_s][K_s] has sizes of its own and
+ * reads rows a_s (one per token): c_s [T][N_s].  act GGB_ACT_NONE (c, c_s fp32) or GGB_ACT_GELU_ERF (both in dt).  A step of few slots
+ * takes one launch. */
+int ggb_op_moe_linear_shared(int dt, const void *w, int64_t N, int64_t K, const void *a, int64_t lda, int gather, int64_t T, int top, int n_exp,
+                             const int32_t *ws, int act, void *c, int64_t ldc, const void *w_s, int64_t N_s, int64_t K_s, const void *a_s, int64_t lda_s,
+                             void *c_s);
 /* Identity experts: the last n_identity of the n_exp experts have no matrices and hand their input through.  Their slots
  * are grouped like the others but no product touches them (w holds n_exp - n_identity experts), and the weighted sum takes
  * the token's row of h (dt, [T][W]: what the experts read) in their place.  moe_linear act 3 (steps of at most 16 slots):
