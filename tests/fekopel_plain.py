@@ -127,11 +127,33 @@ def route(h, router, top, groups=1, keep=1, scale=1.0):
     return order, w / (w.sum(axis=-1, keepdims=True) + 1e-20) * scale
 
 
-def moe_ff(h, W, p, f):
+def route_margin(h, router, top, groups=1, keep=1):
+    """How far in logits the choice of every token is from another one: the last group that stays to the first that goes, the last
+    expert chosen to the first that is not."""
+    z = h @ router.T
+    T, E = z.shape
+    best = z.reshape(T, groups, E // groups).max(axis=-1)
+    order = np.argsort(-best, axis=-1, kind="stable")
+    gap = np.full(T, np.inf)
+    cand = z.reshape(T, groups, E // groups).copy()
+    if keep < groups:
+        rows = np.arange(T)
+        gap = best[rows, order[:, keep - 1]] - best[rows, order[:, keep]]
+        for t in range(T):
+            cand[t, order[t, keep:]] = -np.inf
+    ranked = -np.sort(-cand.reshape(T, E), axis=-1)
+    if top < E:
+        gap = np.minimum(gap, ranked[:, top - 1] - ranked[:, top])
+    return gap
+
+
+def moe_ff(h, W, p, f, margins=None):
     r = f["router"]
     g = r.get("groups") or {}
     count = g.get("count", 1)
     idx, wt = route(h, W[p + "router"], r["top"], count, g.get("keep", count), r.get("scale", 1.0))
+    if margins is not None:
+        margins.append(route_margin(h, W[p + "router"], r["top"], count, g.get("keep", count)))
     out = np.zeros_like(h)
     for e in np.unique(idx):
         t, slot = np.nonzero(idx == e)
@@ -156,8 +178,8 @@ def layer_runs(cfg):
 MIXERS = {"attention": attention_sink, "attention_2": attention_gated}
 
 
-def forward(tokens, W, cfg, layers_out=None):
-    """Logits [T, vocab] of a whole sequence; layers_out collects the residual after every layer run."""
+def forward(tokens, W, cfg, layers_out=None, margins=None):
+    """Logits [T, vocab] of a whole sequence; layers_out collects the residual after every layer run, margins every router's."""
     eps = cfg["norm"]["eps"]
     x0 = W["embed"][np.asarray(tokens)].astype(np.float64)
     x = x0.copy()
@@ -171,7 +193,7 @@ def forward(tokens, W, cfg, layers_out=None):
             x = x + (x0 if step > 0 else 0.0) + W["loop.step"][step]
         x = x + MIXERS[L["type"]](norm(x, p + "norm1"), W, p + "mix.", L["mixer"], eps)
         if L.get("mlp"):
-            x = x + moe_ff(norm(x, p + "norm2"), W, p + "mlp.", L["mlp"])
+            x = x + moe_ff(norm(x, p + "norm2"), W, p + "mlp.", L["mlp"], margins)
         if layers_out is not None:
             layers_out.append(x)
     return norm(x, "final.norm") @ W["head"].T
