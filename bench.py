@@ -1205,13 +1205,104 @@ def run_tezesun(args):
                       "peaks": peaks, "sizes": records}), flush=True)
 
 
+FEKOPEL_SIZES = {  # width, layers, heads, kv heads, head size, window, kept tokens, experts, groups, groups that stay, top, expert ff, shared ff, vocab
+    "s": (1024, 8, 8, 2, 128, 1024, 4, 16, 4, 2, 2, 1024, 1024, 32000),
+    "m": (2048, 8, 16, 4, 128, 1024, 4, 32, 4, 2, 4, 1408, 2816, 32000),
+    "l": (4096, 4, 32, 8, 128, 2048, 4, 16, 4, 2, 2, 2048, 4096, 32000),
+}
+FK_OPS = ("op_linear", "op_attn", "op_attn_prep", "op_act", "op_residual", "op_rows", "op_moe", "op_moe_linear")
+
+
+def fekopel_config(size):
+    """Layers alternate: the gated mixer with positions, then the one with a sink; experts in every layer; the two middle layers run twice."""
+    W, L, H, Gk, D, win, keep, E, groups, stay, top, ff, fs, V = FEKOPEL_SIZES[size]
+    base = {"heads": H, "kv_heads": Gk, "dim": D, "vdim": D, "scale": D ** -0.5}
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": fs}, "router": {"experts": E, "top": top, "scale": 2.0, "groups": {"count": groups, "keep": stay}}}
+    two = dict(base, softcap=30.0, mask={"size": win, "keep_first": keep}, rot={"base": 500000.0, "dims": D // 2})
+    one = dict(base, mask={"size": win})
+    return {"architecture": "Fekopel", "vocab": V, "width": W, "norm": {"eps": 1e-5}, "loop": {"start": L // 2 - 1, "stop": L // 2 + 1, "times": 2},
+            "layers": [{"type": "attention_2", "mixer": two, "mlp": mlp} if i % 2 == 0 else {"type": "attention", "mixer": one, "mlp": mlp} for i in range(L)]}
+
+
+def fekopel_peer_config(size):
+    """The Kibilix model of the same shape: attention in chunks as long as the window, one residual, as many gated experts of the same size
+    with a soft-max router, the same looped layers."""
+    W, L, H, Gk, D, win, keep, E, groups, stay, top, ff, fs, V = FEKOPEL_SIZES[size]
+    mx = {"heads": H, "kv_heads": Gk, "dim": D, "vdim": D, "scale": D ** -0.5, "softcap": 30.0, "mask": {"size": win}, "rot": {"base": 500000.0, "dims": D // 2}}
+    mlp = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": E, "identity": 0, "top": top}}
+    return {"architecture": "Kibilix", "vocab": V, "width": W, "norm": {"eps": 1e-5}, "loop": {"start": L // 2 - 1, "stop": L // 2 + 1, "times": 2},
+            "layers": [{"type": "attention", "mixer": mx, "mlp": mlp}] * L}
+
+
+def _fekopel_record(G, peaks, size, T, ctx, n_dec, peer):
+    W, L, H, Gk, D, win, keep, E, groups, stay, top, ff, fs, V = FEKOPEL_SIZES[size]
+    runs = L + 2
+    eng = G.Engine(config=fekopel_peer_config(size) if peer else fekopel_config(size), seed=7, dtype="bfloat16", max_tokens=ctx + n_dec + 64, page_size=64, max_portion=1024)
+    pf, pf_ops, dec, dc_ops, kernels, clocks = _engine_times(G, eng, V, T, ctx, n_dec, FK_OPS)
+    wbytes = eng.stats()["weight_bytes"]
+    eng.close()
+    # per layer run; a gate per element in every second run of the design itself
+    gate = 0.0 if peer else 0.5 * H * D
+    lin = runs * W * (2.0 * H * D + 2 * Gk * D + gate)
+    exp = runs * W * (top * 3.0 * ff if peer else 2.0 * (top * ff + fs))
+    keys = float(sum(i % win + 1 if peer else min(i + 1, win) for i in range(T)))
+    attn_flops = runs * 4.0 * H * D * keys
+    cache_bytes = runs * 2.0 * 2 * Gk * D * (((ctx - 1) % win + 1) if peer else min(ctx, win))
+    # two passes over the residual per run: x in and out, a mixer's row in and `top` (and the shared) rows in, two bf16 rows out
+    res_bytes = runs * W * (4.0 * (4 + 1 + top + (0 if peer else 1)) + 4.0) * T
+    lin_flops, lin_bytes = 2.0 * T * lin + 2.0 * V * W, 2.0 * (lin + V * W)
+    ms = lambda ops, k: ops[k] / 1e3
+    return {
+        "config": {"width": W, "layers": L, "layer_runs": runs, "heads": H, "kv_heads": Gk, "dim": D, "window": win, "kept": keep, "experts": E, "groups": groups, "stay": stay, "top": top,
+                   "expert_ff": ff, "shared_ff": 0 if peer else fs, "vocab": V, "weight_bytes": wbytes},
+        "prefill": {"tokens": T, "tokens_per_s": T / pf, "ms": 1e3 * pf, "op_ms": pf_ops, "clocks": clocks,
+                    "linear_tflops": lin_flops / ms(pf_ops, "op_linear") / 1e12,
+                    "linear_frac_of_tensor_peak": lin_flops / ms(pf_ops, "op_linear") / 1e12 / peaks["bf16_tflops_sustained"],
+                    "experts_tflops": 2.0 * T * exp / ms(pf_ops, "op_moe_linear") / 1e12,
+                    "experts_frac_of_tensor_peak": 2.0 * T * exp / ms(pf_ops, "op_moe_linear") / 1e12 / peaks["bf16_tflops_sustained"],
+                    "attn_tflops_cuda_cores": attn_flops / ms(pf_ops, "op_attn") / 1e12, "residual_gbs": res_bytes / ms(pf_ops, "op_residual") / 1e9},
+        "decode": {"n_kv": ctx, "tokens_per_s": 1.0 / dec, "us_per_token": 1e6 * dec, "kernels_per_token": kernels, "op_us": {k: 1e3 * v for k, v in dc_ops.items()},
+                   "linear_gbs": lin_bytes / ms(dc_ops, "op_linear") / 1e9, "linear_frac_of_hbm_peak": lin_bytes / ms(dc_ops, "op_linear") / 1e9 / peaks["hbm_gbs"],
+                   "experts_gbs": 2.0 * exp / ms(dc_ops, "op_moe_linear") / 1e9, "attn_gbs": cache_bytes / ms(dc_ops, "op_attn") / 1e9,
+                   "token_frac_of_hbm_roofline": ((lin_bytes + 2.0 * exp + cache_bytes) / (peaks["hbm_gbs"] * 1e9)) / dec},
+    }
+
+
+def run_fekopel(args):
+    """--arch fekopel: prefill and decode throughput of the Fekopel design (random bf16 weights) at layer sizes of real models, through the
+    serving engine (host call: H2D token ids, operator launches / graph replay, D2H result), with cudaEvent time per operator class
+    and roofline fractions; beside it the closest model of the framework, Kibilix with attention layers only, at the same width,
+    depth, loop, heads, experts and expert size."""
+    import gemma_ggml_b200 as G
+    G.init(0)
+    peaks = {"hbm_gbs": 6650.0, "bf16_tflops_sustained": 1400.0, "source": "fallback"}
+    try:
+        pk = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
+        peaks = {"hbm_gbs": float(pk["hbm_gbs"]), "bf16_tflops_sustained": float(pk["bf16_tflops_sustained"]), "source": "MEASURED_PEAKS.json"}
+    except Exception:
+        pass
+    T, ctx, n_dec = args.prefill_tokens if args.prefill_tokens != 512 else 2048, args.ctx, min(args.steps, 128)
+    records = {}
+    for size in args.sizes.split(","):
+        records[size] = _fekopel_record(G, peaks, size, T, ctx, n_dec, False)
+        if not args.no_sub_records:
+            records[size]["kibilix_equal_size"] = _fekopel_record(G, peaks, size, T, ctx, n_dec, True)
+    first = records[args.sizes.split(",")[0]]
+    print(json.dumps({"metric": "fekopel decode tokens/s", "value": first["decode"]["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+                      "steps": n_dec, "warmup": 8, "ms_per_step": first["decode"]["us_per_token"] / 1e3, "higher_is_better": True,
+                      "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic (random bf16 weights of the configured sizes)",
+                      "config": {"workload": "Fekopel sizes " + args.sizes + ": prefill of %d tokens, greedy decode at n_kv %d, through the serving engine" % (T, ctx),
+                                 "l2": "weights of every size exceed the 126 MB L2"},
+                      "peaks": peaks, "sizes": records}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--arch", default="gemma", choices=["gemma", "safolorn", "begupel", "ditalorn", "kibilix", "tezesun"],
+    ap.add_argument("--arch", default="gemma", choices=["gemma", "safolorn", "begupel", "ditalorn", "kibilix", "tezesun", "fekopel"],
                     help="gemma: the headline workload (default); safolorn: throughput of the Safolorn design beside Gemma at equal size; "
                          "begupel: throughput of the Begupel design beside Safolorn at equal size; ditalorn: the Ditalorn design beside Safolorn at equal size; kibilix: the Kibilix design beside Begupel at equal size; "
-                         "tezesun: the Tezesun design beside Begupel and Safolorn at equal size")
-    ap.add_argument("--sizes", default="s,m,l", help="--arch safolorn / begupel / ditalorn / kibilix / tezesun: which of the sizes s, m, l to run")
+                         "tezesun: the Tezesun design beside Begupel and Safolorn at equal size; fekopel: the Fekopel design beside Kibilix at equal size")
+    ap.add_argument("--sizes", default="s,m,l", help="--arch safolorn / begupel / ditalorn / kibilix / tezesun / fekopel: which of the sizes s, m, l to run")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=256)
     ap.add_argument("--warmup", type=int, default=16)
@@ -1239,6 +1330,8 @@ def main():
         run_kibilix(args)
     elif args.arch == "tezesun":
         run_tezesun(args)
+    elif args.arch == "fekopel":
+        run_fekopel(args)
     elif args.mode == "prefill":
         run_prefill(args)
     else:
