@@ -17,13 +17,17 @@ template <typename E>
 __device__ __forceinline__ float router_dot(const E *__restrict__ hr, const float *__restrict__ wr, int64_t W, int lane) {
     float s = 0.f;
     if (W % 4 == 0) {
-#pragma unroll 4
+        struct alignas(4 * sizeof(E)) quad { // four numbers in one load: rows of a multiple of four are aligned to it
+            E v[4];
+        };
+#pragma unroll 8
         for (int64_t k = (int64_t)lane * 4; k < W; k += 128) {
             const float4 wv = *reinterpret_cast<const float4 *>(wr + k);
-            s = fmaf(wv.x, to_f32(hr[k]), s);
-            s = fmaf(wv.y, to_f32(hr[k + 1]), s);
-            s = fmaf(wv.z, to_f32(hr[k + 2]), s);
-            s = fmaf(wv.w, to_f32(hr[k + 3]), s);
+            const quad hv = *reinterpret_cast<const quad *>(hr + k);
+            s = fmaf(wv.x, to_f32(hv.v[0]), s);
+            s = fmaf(wv.y, to_f32(hv.v[1]), s);
+            s = fmaf(wv.z, to_f32(hv.v[2]), s);
+            s = fmaf(wv.w, to_f32(hv.v[3]), s);
         }
     } else {
         for (int64_t k = lane; k < W; k += 32) s = fmaf(wr[k], to_f32(hr[k]), s);
