@@ -1247,13 +1247,14 @@ def _fekopel_record(G, peaks, size, T, ctx, n_dec, peer):
     exp = runs * W * (top * 3.0 * ff if peer else 2.0 * (top * ff + fs))
     keys = float(sum(i % win + 1 if peer else min(i + 1, win) for i in range(T)))
     attn_flops = runs * 4.0 * H * D * keys
-    cache_bytes = runs * 2.0 * 2 * Gk * D * (((ctx - 1) % win + 1) if peer else min(ctx, win))
+    pos = ctx + n_dec + 16  # where the profiled steps are: a chunk has begun anew shortly before, a window is full
+    cache_bytes = runs * 2.0 * 2 * Gk * D * (pos % win + 1 if peer else min(pos, win))
     # two passes over the residual per run: x in and out, a mixer's row in and `top` (and the shared) rows in, two bf16 rows out
     res_bytes = runs * W * (4.0 * (4 + 1 + top + (0 if peer else 1)) + 4.0) * T
     lin_flops, lin_bytes = 2.0 * T * lin + 2.0 * V * W, 2.0 * (lin + V * W)
     ms = lambda ops, k: ops[k] / 1e3
     return {
-        "config": {"width": W, "layers": L, "layer_runs": runs, "heads": H, "kv_heads": Gk, "dim": D, "window": win, "kept": keep, "experts": E, "groups": groups, "stay": stay, "top": top,
+        "config": {"width": W, "layers": L, "layer_runs": runs, "decode_keys": pos % win + 1 if peer else min(pos, win), "heads": H, "kv_heads": Gk, "dim": D, "window": win, "kept": keep, "experts": E, "groups": groups, "stay": stay, "top": top,
                    "expert_ff": ff, "shared_ff": 0 if peer else fs, "vocab": V, "weight_bytes": wbytes},
         "prefill": {"tokens": T, "tokens_per_s": T / pf, "ms": 1e3 * pf, "op_ms": pf_ops, "clocks": clocks,
                     "linear_tflops": lin_flops / ms(pf_ops, "op_linear") / 1e12,
